@@ -101,13 +101,22 @@ void gather_rows(const at::Tensor& x, const at::Tensor& idx, at::Tensor out) {
 }
 
 // impl: 0 = tcgen05, 1 = SIMT reference
+// [lam, post, eps, dv] -> the kernels' parameters (empty: not differential)
+sglb::DiffCombine diff_combine(const std::vector<double>& a) {
+  sglb::DiffCombine d;
+  if (a.empty()) return d;
+  TORCH_CHECK(a.size() == 4, "differential attention takes [lam, post, eps, dv]");
+  d.lam = (float)a[0]; d.post = (float)a[1]; d.eps = (float)a[2]; d.dv = (int)a[3];
+  return d;
+}
+
 void attn_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor out,
               c10::optional<at::Tensor> lse, c10::optional<at::Tensor> part_o, c10::optional<at::Tensor> part_lse,
               const at::Tensor& page_table, const at::Tensor& req_slots, const at::Tensor& seq_lens,
               c10::optional<at::Tensor> cu_q, c10::optional<at::Tensor> tok2req, int64_t max_q_len, int64_t page_size,
               int64_t num_splits, double scale, bool causal, int64_t window, double logit_cap, double k_scale,
               double v_scale, int64_t impl, c10::optional<at::Tensor> tree_anc, c10::optional<at::Tensor> slopes,
-              c10::optional<at::Tensor> log_rates, int64_t keep_first) {
+              c10::optional<at::Tensor> log_rates, int64_t keep_first, int64_t chunk, std::vector<double> diff_args) {
   CHECK_CUDA(q); CHECK_BF16(q); CHECK_BF16(out); CHECK_I32(page_table); CHECK_I32(req_slots); CHECK_I32(seq_lens);
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2), "q must be [T, Hq, D] with packed heads");
   TORCH_CHECK(k_cache.dim() == 3 && v_cache.dim() == 3, "k_cache must be [slots, Hkv, D]");
@@ -115,6 +124,11 @@ void attn_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& 
   const bool tc_impl = impl == 0 || impl == 2;
   const bool rows_ok = k_cache.stride(2) == 1 && k_cache.stride(1) == k_cache.size(2) && v_cache.strides() == k_cache.strides() &&
                        k_cache.stride(0) >= k_cache.size(1) * k_cache.size(2);
+  // differential form: diff = [lam, post, eps, dv], out [T, Hq / 2, dv]
+  const sglb::DiffCombine dc = diff_combine(diff_args);
+  const sglb::DiffCombine* diff = diff_args.empty() ? nullptr : &dc;
+  TORCH_CHECK(out.numel() == (diff ? q.size(0) * (q.size(1) / 2) * dc.dv : q.numel()), "attn_fwd: out size");
+  TORCH_CHECK((chunk <= 0 && !diff) || (tc_impl && causal && !tree_anc.has_value()), "attn_fwd: chunks and the differential form need the tcgen05 kernels, causal");
   TORCH_CHECK(out.is_contiguous() && (tc_impl ? rows_ok : (k_cache.is_contiguous() && v_cache.is_contiguous())), "attn_fwd: cache layout");
   const int kv_stride = (int)k_cache.stride(0);
   const int T = (int)q.size(0), Hq = (int)q.size(1), D = (int)q.size(2), Hkv = (int)k_cache.size(1);
@@ -154,7 +168,7 @@ void attn_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& 
                            opt_mptr<float>(part_lse), page_table.data_ptr<int>(), (int)page_table.stride(0), req_slots.data_ptr<int>(),
                            seq_lens.data_ptr<int>(), B, (int)q.stride(0), Hq, Hkv, D, (int)k_cache.size(0), (int)page_size, (int)num_splits,
                            (float)scale, (int)window, (float)logit_cap, sched_ptr, num_sms(), cur_stream(), opt_ptr<float>(slopes), opt_ptr<float>(log_rates),
-                           (int)keep_first, kv_stride);
+                           (int)keep_first, kv_stride, (int)chunk, diff);
       count(num_splits > 1 ? 2 : 1);
       return;
     }
@@ -165,7 +179,7 @@ void attn_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& 
                       (int)q.stride(0), (int)max_q_len, Hq, Hkv, D, (int)k_cache.size(0), (int)page_size, (int)num_splits,
                       (float)scale, causal ? 1 : 0, (int)window, (float)logit_cap, sched_ptr, num_sms(), cur_stream(),
                       tree_anc.has_value() ? reinterpret_cast<const unsigned*>(tree_anc->data_ptr<int>()) : nullptr, opt_ptr<float>(slopes),
-                      opt_ptr<float>(log_rates), (int)keep_first, kv_stride);
+                      opt_ptr<float>(log_rates), (int)keep_first, kv_stride, (int)chunk, diff);
     count(num_splits > 1 ? 2 : 1);
   } else {
     TORCH_CHECK(!tree_anc.has_value(), "tree masks need the tcgen05 attention (impl 0 / 2)");
@@ -399,12 +413,17 @@ void qk_norm_cache_write(const at::Tensor& qkv, int64_t H, int64_t G, int64_t D,
 void window_attention(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, int64_t G, int64_t Dv, const at::Tensor& page_table,
                       const at::Tensor& req_slots, const at::Tensor& seq_lens, c10::optional<at::Tensor> cu_q, int64_t max_q_len, int64_t page_size,
                       double scale, double softcap, int64_t window, c10::optional<at::Tensor> slopes, c10::optional<at::Tensor> sinks, at::Tensor out,
-                      int64_t dim, int64_t pad, int64_t keep_first, c10::optional<at::Tensor> log_rates, c10::optional<at::Tensor> gate, double out_scale) {
+                      int64_t dim, int64_t pad, int64_t keep_first, c10::optional<at::Tensor> log_rates, c10::optional<at::Tensor> gate, double out_scale,
+                      int64_t chunk, std::vector<double> diff_args) {
+  const sglb::DiffCombine dc = diff_combine(diff_args);
+  const sglb::DiffCombine* diff = diff_args.empty() ? nullptr : &dc;
+  const int64_t Ho = diff ? q.size(1) / 2 : q.size(1);          // output heads: the differential form combines pairs of query heads
+  TORCH_CHECK(!diff || (q.size(1) % 2 == 0 && dc.dv == Dv && !gate.has_value() && !sinks.has_value() && !slopes.has_value()));
   CHECK_CUDA(q); CHECK_I32(page_table); CHECK_I32(req_slots); CHECK_I32(seq_lens);
   // out: [T, H, Dv] contiguous, or a [T, H * Dv] block of columns of a wider buffer
-  TORCH_CHECK(bf16_or_f32(q) && q.dim() == 3 && q.is_contiguous() && out.scalar_type() == q.scalar_type() && out.numel() == q.size(0) * q.size(1) * Dv &&
-              (out.is_contiguous() || (out.dim() == 2 && out.stride(1) == 1 && out.size(1) == q.size(1) * Dv)));
-  const int ldo = out.dim() == 2 ? (int)out.stride(0) : (int)(q.size(1) * Dv);
+  TORCH_CHECK(bf16_or_f32(q) && q.dim() == 3 && q.is_contiguous() && out.scalar_type() == q.scalar_type() && out.numel() == q.size(0) * Ho * Dv &&
+              (out.is_contiguous() || (out.dim() == 2 && out.stride(1) == 1 && out.size(1) == Ho * Dv)));
+  const int ldo = out.dim() == 2 ? (int)out.stride(0) : (int)(Ho * Dv);
   // pad > 0: q [T, H, pad] and every key / value head occupy ``pad`` columns of which the first ``dim`` / ``Dv`` count
   const int64_t H = q.size(1), D = pad > 0 ? dim : q.size(2);
   TORCH_CHECK(pad == 0 || (q.size(2) == pad && D >= 1 && D <= pad && Dv <= pad));
@@ -429,7 +448,72 @@ void window_attention(const at::Tensor& q, const at::Tensor& k_cache, const at::
                          seq_lens.data_ptr<int>(), opt_ptr<int>(cu_q), B, cu_q.has_value() ? (int)max_q_len : 1, (float)scale, (float)softcap, (int)window,
                          opt_ptr<float>(slopes), opt_ptr<float>(sinks), out.data_ptr(), (int)pad, (int)keep_first, opt_ptr<float>(log_rates),
                          gate.has_value() ? gate->data_ptr() : nullptr, gate.has_value() ? (int)gate->stride(0) : 0, gate_per_head, ldo, (float)out_scale,
-                         cur_stream());
+                         (int)chunk, diff, cur_stream());
+  count();
+}
+
+void conv_attention_prepare(const at::Tensor& qkv, int64_t H, int64_t G, int64_t M, int64_t D, int64_t Dv, const at::Tensor& conv_w, at::Tensor conv_state,
+                            const at::Tensor& positions, c10::optional<at::Tensor> cu_q, const at::Tensor& req_slots, const at::Tensor& seq_lens,
+                            c10::optional<at::Tensor> q_norm_w, c10::optional<at::Tensor> k_norm_w, double eps, c10::optional<at::Tensor> inv_freq,
+                            double rot_mult, at::Tensor k_cache, at::Tensor v_cache, const at::Tensor& loc, at::Tensor q_out, int64_t pad) {
+  CHECK_CUDA(qkv); CHECK_I32(positions); CHECK_I32(loc); CHECK_I32(req_slots); CHECK_I32(seq_lens);
+  const int64_t T = qkv.size(0), C = (H + G) * M * D + G * Dv, taps = conv_w.size(1);
+  auto same = [&](const at::Tensor& t) { return t.scalar_type() == qkv.scalar_type(); };
+  TORCH_CHECK(bf16_or_f32(qkv) && qkv.dim() == 2 && qkv.stride(1) == 1 && qkv.size(1) >= C && H >= 1 && G >= 1 && M >= 1 && H % G == 0 && D >= 1 && Dv >= 1);
+  TORCH_CHECK(same(conv_w) && conv_w.is_contiguous() && conv_w.size(0) == C && same(conv_state) && conv_state.is_contiguous() && conv_state.dim() == 3 &&
+              (taps == 1 || (conv_state.size(1) == C && conv_state.size(2) == taps - 1)), "conv_attention_prepare: taps [C, K], state [slots, C, K - 1]");
+  TORCH_CHECK(pad == 0 || (pad % M == 0 && D <= pad / M && Dv <= pad));
+  const int64_t seg = pad > 0 ? pad / M : D, wv = pad > 0 ? pad : Dv;
+  TORCH_CHECK(same(q_out) && q_out.is_contiguous() && q_out.numel() == T * H * M * M * seg);
+  TORCH_CHECK(same(k_cache) && same(v_cache) && k_cache.dim() == 3 && k_cache.size(1) == 1 && k_cache.stride(2) == 1 && v_cache.stride(2) == 1 &&
+              k_cache.stride(0) == v_cache.stride(0) && k_cache.size(2) >= G * M * seg && v_cache.size(2) >= G * wv && positions.numel() == T && loc.numel() == T);
+  TORCH_CHECK(q_norm_w.has_value() == k_norm_w.has_value());
+  if (q_norm_w.has_value())
+    TORCH_CHECK(same(*q_norm_w) && same(*k_norm_w) && q_norm_w->is_contiguous() && k_norm_w->is_contiguous() && q_norm_w->numel() == D && k_norm_w->numel() == D);
+  int half = 0;
+  if (inv_freq.has_value()) {
+    TORCH_CHECK(inv_freq->scalar_type() == at::kFloat && inv_freq->is_contiguous() && 2 * inv_freq->numel() <= D);
+    half = (int)inv_freq->numel();
+  }
+  const int B = (int)req_slots.size(0);
+  TORCH_CHECK(seq_lens.numel() == B);
+  if (cu_q.has_value()) { CHECK_I32(*cu_q); TORCH_CHECK(cu_q->numel() == B + 1); } else TORCH_CHECK(T == B);
+  if (T == 0) return;
+  c10::cuda::CUDAGuard g(qkv.device());
+  sglb::conv_attention_prepare(qkv.data_ptr(), (int)qkv.stride(0), qkv.scalar_type() == at::kBFloat16, (int)T, (int)H, (int)G, (int)M, (int)D, (int)Dv,
+                               conv_w.data_ptr(), (int)taps, conv_state.data_ptr(), positions.data_ptr<int>(), opt_ptr<int>(cu_q), req_slots.data_ptr<int>(),
+                               seq_lens.data_ptr<int>(), B, q_norm_w.has_value() ? q_norm_w->data_ptr() : nullptr,
+                               k_norm_w.has_value() ? k_norm_w->data_ptr() : nullptr, (float)eps, half > 0 ? inv_freq->data_ptr<float>() : nullptr, half,
+                               (float)rot_mult, k_cache.data_ptr(), v_cache.data_ptr(), (size_t)k_cache.stride(0), loc.data_ptr<int>(), q_out.data_ptr(),
+                               (int)pad, num_sms(), cur_stream());
+  count(cu_q.has_value() && taps > 1 ? 2 : 1);
+}
+
+void norm_add_f32(at::Tensor x, const at::Tensor& src, c10::optional<at::Tensor> ids, const at::Tensor& w, c10::optional<at::Tensor> out, double eps,
+                  bool zero_centred) {
+  CHECK_CUDA(x);
+  TORCH_CHECK(x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous() && src.dim() == 2 && src.is_contiguous() && bf16_or_f32(src) &&
+              src.size(1) == x.size(1) && bf16_or_f32(w) && w.is_contiguous() && w.numel() == x.size(1));
+  if (ids.has_value()) { CHECK_I32(*ids); TORCH_CHECK(ids->is_contiguous() && ids->numel() == x.size(0) && src.size(0) >= 1); }
+  else TORCH_CHECK(src.size(0) == x.size(0));
+  if (out.has_value()) TORCH_CHECK(out->scalar_type() == w.scalar_type() && out->is_contiguous() && out->numel() == x.numel());
+  if (x.size(0) == 0) return;
+  c10::cuda::CUDAGuard g(x.device());
+  sglb::norm_add_f32(x.data_ptr<float>(), src.data_ptr(), src.scalar_type() == at::kBFloat16, opt_ptr<int>(ids), (int)src.size(0), w.data_ptr(),
+                     out.has_value() ? out->data_ptr() : nullptr, w.scalar_type() == at::kBFloat16, (int)x.size(0), (int)x.size(1), (float)eps, zero_centred,
+                     cur_stream());
+  count();
+}
+
+void moe_sigmoid_route(const at::Tensor& logits, bool renorm, double scale, at::Tensor w, at::Tensor ids) {
+  CHECK_CUDA(logits); CHECK_I32(ids);
+  const int64_t T = logits.size(0), K = w.size(1);
+  TORCH_CHECK(logits.scalar_type() == at::kFloat && logits.dim() == 2 && logits.stride(1) == 1 && w.scalar_type() == at::kFloat && w.is_contiguous() &&
+              ids.is_contiguous() && w.size(0) == T && ids.size(0) == T && ids.size(1) == K);
+  if (T == 0) return;
+  c10::cuda::CUDAGuard g(logits.device());
+  sglb::moe_sigmoid_route(logits.data_ptr<float>(), (int)logits.stride(0), (int)T, (int)logits.size(1), (int)K, renorm, (float)scale, w.data_ptr<float>(),
+                          ids.data_ptr<int>(), cur_stream());
   count();
 }
 
@@ -1006,16 +1090,17 @@ void moe_topk_softmax(const at::Tensor& logits, at::Tensor out_w, at::Tensor out
 }
 
 // Whole expert MLP block on expert-sorted rows: align -> gather -> grouped GEMM (silu(gate)*up fused) -> grouped GEMM (routing
-// weight fused) -> combine.  With peer pointers the combine pushes its result into every peer's NVLink arena instead of `out`.
+// weight fused) -> combine.  act: 0 = silu(gate) * up, 1 = clamped GLU, 2 = ungated max(up, 0)^2 (w13 = [E, I, H]).  ``weight_input``: the routing weight
+// multiplies an expert's input (in the gather) instead of its output.  With peer pointers the combine pushes its result into every peer's NVLink arena instead of `out`.
 void moe_grouped_mlp_impl(const at::Tensor& x, const at::Tensor& w13, const at::Tensor& w2, const at::Tensor& topk_w,
                           const at::Tensor& topk_ids, c10::optional<at::Tensor> out, int64_t expert_offset,
                           const int64_t* peer_slots, const int64_t* peer_flags, int rank, int world, const uint32_t* epoch,
-                          uint32_t* done, int act = 0, float act_limit = 0.f, float act_alpha = 0.f) {
+                          uint32_t* done, int act = 0, float act_limit = 0.f, float act_alpha = 0.f, bool weight_input = false) {
   CHECK_CUDA(x); CHECK_BF16(x); CHECK_BF16(w13); CHECK_BF16(w2); CHECK_I32(topk_ids); CHECK_LAST_CONTIG(x);
   TORCH_CHECK(x.dim() == 2 && w13.dim() == 3 && w2.dim() == 3 && w13.is_contiguous() && w2.is_contiguous());
   TORCH_CHECK(topk_w.scalar_type() == at::kFloat && topk_w.is_contiguous() && topk_ids.is_contiguous());
   const int T = (int)x.size(0), H = (int)x.size(1), K = (int)topk_ids.size(1), E = (int)w13.size(0), I = (int)w2.size(2);
-  TORCH_CHECK(w13.size(1) == 2 * I && w13.size(2) == H && w2.size(1) == H && w2.size(0) == E);
+  TORCH_CHECK(w13.size(1) == (act == 2 ? I : 2 * I) && w13.size(2) == H && w2.size(1) == H && w2.size(0) == E);
   if (T == 0) return;
   c10::cuda::CUDAGuard g(x.device());
   auto stream = cur_stream();
@@ -1032,11 +1117,15 @@ void moe_grouped_mlp_impl(const at::Tensor& x, const at::Tensor& w13, const at::
   sglb::moe_align(topk_ids.data_ptr<int>(), topk_w.data_ptr<float>(), pairs, E, (int)expert_offset, sorted_row, inv_pos,
                   row_w.data_ptr<float>(), tile_expert, num_tiles, max_tiles, stream);
   auto xs = at::empty({cap, H}, x.options());
-  sglb::moe_gather(x.data_ptr(), sorted_row, num_tiles, xs.data_ptr(), H, (int)x.stride(0), K, cap, num_sms(), stream);
+  sglb::moe_gather(x.data_ptr(), sorted_row, num_tiles, xs.data_ptr(), H, (int)x.stride(0), K, cap, num_sms(), stream,
+                   weight_input ? row_w.data_ptr<float>() : nullptr);
   auto h = at::empty({cap, I}, x.options());
   if (act == 0) {
     sglb::gemm_bf16_tc_grouped(xs.data_ptr(), w13.data_ptr(), h.data_ptr(), nullptr, cap, I, H, H, I, E, tile_expert, num_tiles, true,
                                num_sms(), stream);
+  } else if (act == 2) {
+    sglb::gemm_bf16_tc_grouped(xs.data_ptr(), w13.data_ptr(), h.data_ptr(), nullptr, cap, I, H, H, I, E, tile_expert, num_tiles, false, num_sms(), stream,
+                               true);
   } else {
     // clamped GLU: the gate|up block comes out of the grouped GEMM whole, the activation is its own (vectorised) pass
     auto h2 = at::empty({cap, 2 * I}, x.options());
@@ -1046,8 +1135,8 @@ void moe_grouped_mlp_impl(const at::Tensor& x, const at::Tensor& w13, const at::
     count();
   }
   auto& ys = xs;   // the gathered inputs are dead once the first GEMM has run (same stream): reuse as the [cap, H] output
-  sglb::gemm_bf16_tc_grouped(h.data_ptr(), w2.data_ptr(), ys.data_ptr(), row_w.data_ptr<float>(), cap, H, I, I, H, E, tile_expert,
-                             num_tiles, false, num_sms(), stream);
+  sglb::gemm_bf16_tc_grouped(h.data_ptr(), w2.data_ptr(), ys.data_ptr(), weight_input ? nullptr : row_w.data_ptr<float>(), cap, H, I, I, H, E,
+                             tile_expert, num_tiles, false, num_sms(), stream);
   if (peer_slots) {
     sglb::moe_combine_push(ys.data_ptr(), inv_pos, nullptr, T, H, K, peer_slots, peer_flags, rank, world, epoch, done, num_sms(), stream);
   } else {
@@ -1067,6 +1156,12 @@ void moe_grouped_mlp_glu(const at::Tensor& x, const at::Tensor& w13, const at::T
                          const at::Tensor& topk_ids, at::Tensor out, int64_t expert_offset, double limit, double alpha) {
   CHECK_BF16(out);
   moe_grouped_mlp_impl(x, w13, w2, topk_w, topk_ids, out, expert_offset, nullptr, nullptr, 0, 1, nullptr, nullptr, 1, (float)limit, (float)alpha);
+}
+
+void moe_grouped_mlp_relu2(const at::Tensor& x, const at::Tensor& w1, const at::Tensor& w2, const at::Tensor& topk_w, const at::Tensor& topk_ids,
+                           at::Tensor out, int64_t expert_offset, bool weight_input) {
+  CHECK_BF16(out);
+  moe_grouped_mlp_impl(x, w1, w2, topk_w, topk_ids, out, expert_offset, nullptr, nullptr, 0, 1, nullptr, nullptr, 2, 0.f, 0.f, weight_input);
 }
 
 void moe_grouped_mlp_push(const at::Tensor& x, const at::Tensor& w13, const at::Tensor& w2, const at::Tensor& topk_w,
@@ -1126,7 +1221,8 @@ TORCH_LIBRARY(sglb, m) {
   m.def("attn_fwd(Tensor q, Tensor k_cache, Tensor v_cache, Tensor(a!) out, Tensor(b!)? lse, Tensor(c!)? part_o, "
         "Tensor(d!)? part_lse, Tensor page_table, Tensor req_slots, Tensor seq_lens, Tensor? cu_q, Tensor? tok2req, "
         "int max_q_len, int page_size, int num_splits, float scale, bool causal, int window, float logit_cap, "
-        "float k_scale, float v_scale, int impl, Tensor? tree_anc=None, Tensor? slopes=None, Tensor? log_rates=None, int keep_first=0) -> ()", &attn_fwd);
+        "float k_scale, float v_scale, int impl, Tensor? tree_anc=None, Tensor? slopes=None, Tensor? log_rates=None, int keep_first=0, int chunk=0, "
+        "float[] diff=[]) -> ()", &attn_fwd);
   m.def("attn_decode_prof(Tensor buf) -> ()", &attn_decode_prof);
   m.def("green_ctx_streams(int device, int[] sm_counts) -> int[]", [](int64_t device, std::vector<int64_t> counts) {
     std::vector<long long> c(counts.begin(), counts.end());
@@ -1153,8 +1249,15 @@ TORCH_LIBRARY(sglb, m) {
         "Tensor(a!) k_cache, Tensor(b!) v_cache, Tensor loc, bool normalise, Tensor(c!) q_out, int pad=0) -> ()", &qk_norm_cache_write);
   m.def("window_attention(Tensor q, Tensor k_cache, Tensor v_cache, int G, int Dv, Tensor page_table, Tensor req_slots, Tensor seq_lens, Tensor? cu_q, "
         "int max_q_len, int page_size, float scale, float softcap, int window, Tensor? slopes, Tensor? sinks, Tensor(a!) out, int dim, int pad=0, "
-        "int keep_first=0, Tensor? log_rates=None, Tensor? gate=None, float out_scale=1.0) -> ()",
+        "int keep_first=0, Tensor? log_rates=None, Tensor? gate=None, float out_scale=1.0, int chunk=0, float[] diff=[]) -> ()",
         &window_attention);
+  m.def("conv_attention_prepare(Tensor qkv, int H, int G, int M, int D, int Dv, Tensor conv_w, Tensor(a!) conv_state, Tensor positions, Tensor? cu_q, "
+        "Tensor req_slots, Tensor seq_lens, Tensor? q_norm_w, Tensor? k_norm_w, float eps, Tensor? inv_freq, float rot_mult, Tensor(b!) k_cache, "
+        "Tensor(c!) v_cache, Tensor loc, Tensor(d!) q_out, int pad=0) -> ()", &conv_attention_prepare);
+  m.def("norm_add_f32(Tensor(a!) x, Tensor src, Tensor? ids, Tensor w, Tensor(b!)? out, float eps, bool zero_centred=True) -> ()", &norm_add_f32);
+  m.def("moe_sigmoid_route(Tensor logits, bool renorm, float scale, Tensor(a!) w, Tensor(b!) ids) -> ()", &moe_sigmoid_route);
+  m.def("moe_grouped_mlp_relu2(Tensor x, Tensor w1, Tensor w2, Tensor topk_w, Tensor topk_ids, Tensor(a!) out, int expert_offset, bool weight_input) -> ()",
+        &moe_grouped_mlp_relu2);
   m.def("attention_sink_gate(Tensor o, Tensor lse, Tensor sinks, int Dv, Tensor(a!) out) -> ()", &attention_sink_gate);
   m.def("moe_softmax_bias_route(Tensor logits, Tensor? corr, int n_real, Tensor(a!) w, Tensor(b!) ids, Tensor(c!) ident) -> ()", &moe_softmax_bias_route);
   m.def("moe_identity_shared_combine(Tensor(a!) y, Tensor h, Tensor? ident, Tensor? shared, Tensor? gate) -> ()", &moe_identity_shared_combine);

@@ -5,6 +5,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "params.h"
+
 namespace sglb {
 
 // elementwise.cu
@@ -34,13 +36,13 @@ void attn_decode_tc(const void* q, const void* k_cache, const void* v_cache, voi
                     const int* page_table, int pt_stride, const int* req_slots, const int* seq_lens, int B, int q_stride, int Hq, int Hkv,
                     int D, int num_slots, int page_size, int num_splits, float scale, int window, float logit_cap, int* sched, int num_sms,
                     cudaStream_t stream, const float* slopes = nullptr, const float* log_rates = nullptr, int keep_first = 0,
-                    int kv_stride = 0);
+                    int kv_stride = 0, int chunk = 0, const DiffCombine* diff = nullptr);
 void attn_fwd_tc(const void* q, const void* k_cache, const void* v_cache, void* out, float* lse, float* part_o,
                  float* part_lse, const int* page_table, int pt_stride, const int* req_slots, const int* seq_lens,
                  const int* cu_q, int B, int T, int q_stride, int max_q_len, int Hq, int Hkv, int D, int num_slots,
                  int page_size, int num_splits, float scale, int causal, int window, float logit_cap, int* sched, int num_sms,
                  cudaStream_t stream, const unsigned* tree_anc = nullptr, const float* slopes = nullptr, const float* log_rates = nullptr,
-                 int keep_first = 0, int kv_stride = 0);
+                 int keep_first = 0, int kv_stride = 0, int chunk = 0, const DiffCombine* diff = nullptr);
 
 // gemm_tc.cu
 void gemm_bf16_tc(const void* A, const void* W, void* C, const void* bias, int M, int N, int K, int lda, int ldw, int ldc,
@@ -48,7 +50,7 @@ void gemm_bf16_tc(const void* A, const void* W, void* C, const void* bias, int M
 int gemm_pick_bn(int M, int N, int K, int num_sms);
 void gemm_bf16_tc_grouped(const void* A, const void* W, void* C, const float* row_scale, int M_cap, int n_out, int K, int lda,
                           int ldc, int num_experts, const int* tile_expert, const int* num_m_tiles, bool split_silu, int num_sms,
-                          cudaStream_t stream);
+                          cudaStream_t stream, bool relu2 = false);
 
 // kvio.cu: device pool <-> pinned host pool page movers (HiCache L1 <-> L2), zero-copy over UVA, layer_first / page_first host layouts
 void kv_transfer_pages(void* dev, void* host_devptr, const int* dev_pages, const int* host_pages, int n, int planes, long long dev_plane_stride,
@@ -83,7 +85,7 @@ void moe_topk_softmax(const void* logits, bool bf16, float* out_w, int* out_ids,
 void moe_align(const int* topk_ids, const float* topk_w, int n_pairs, int E, int expert_offset, int* sorted_row, int* inv_pos,
                float* row_w, int* tile_expert, int* num_tiles, int max_tiles, cudaStream_t stream);
 void moe_gather(const void* x, const int* sorted_row, const int* num_tiles, void* xs, int H, int x_stride, int K, int cap_rows,
-                int num_sms, cudaStream_t stream);
+                int num_sms, cudaStream_t stream, const float* row_w = nullptr);
 void moe_combine(const void* ys, const int* inv_pos, const float* pair_w, void* out, int T, int H, int K, int num_sms,
                  cudaStream_t stream);
 void moe_combine_push(const void* ys, const int* inv_pos, const float* pair_w, int T, int H, int K, const int64_t* peer_slot_ptrs,
@@ -96,6 +98,8 @@ void sample(const void* logits, bool bf16, int B, int V, int stride, const float
             int* out_tokens, float* out_logprobs, unsigned long long global_seed, const long long* step_ptr, long long step,
             cudaStream_t stream);
 // mamba.cu
+void causal_conv1d_state(const void* x, int ldx, void* conv_state, const int* cu_q, const int* req_slots, const int* seq_lens, int B, int C, int K,
+                         bool bf16, cudaStream_t stream);
 void causal_conv1d(const void* x, int ldx, const void* w, const void* bias, void* conv_state, const int* cu_q, const int* req_slots,
                    const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, float* u, int ldu, cudaStream_t stream);
 void selective_state_update(float* state, const int* req_slots, const float* x, int ldx, const float* dt, const float* A, const float* Bm,
@@ -116,7 +120,7 @@ void qk_norm_cache_write(const void* qkv, int ld, bool bf16, int T, int H, int G
 void window_attention(const void* q, const void* kc, const void* vc, bool bf16, size_t ldc, int H, int G, int D, int Dv, const int* page_table,
                       int pt_stride, int page_size, const int* req_slots, const int* seq_lens, const int* cu_q, int B, int max_q_len, float scale,
                       float softcap, int window, const float* slopes, const float* sinks, void* out, int pad, int keep_first, const float* log_rates,
-                      const void* gate, int ldg, bool gate_per_head, int ldo, float out_scale, cudaStream_t stream);
+                      const void* gate, int ldg, bool gate_per_head, int ldo, float out_scale, int chunk, const DiffCombine* diff, cudaStream_t stream);
 void sigmoid_gate(const void* o, int head_stride, const void* gate, int ldg, bool per_head, bool bf16, int T, int H, int Dv, float scale, void* out, int ldo,
                   cudaStream_t stream);
 void attention_prepare(const void* qkv, int ld, bool bf16, int T, int H, int G, int D, int Dv, const int* positions, const void* q_norm_w, const void* k_norm_w,
@@ -140,6 +144,8 @@ void mamba1_scan(const float* u, const float* dt_raw, int lddt, const float* dt_
 void activation(const void* x, int ldx, bool x_bf16, void* out, bool out_bf16, int T, int n, int act, const void* mul, int ldm, cudaStream_t stream);
 void postnorm_add_rmsnorm_f32(float* residual, const void* delta, bool delta_bf16, const void* post_w, const void* w, void* out, bool out_bf16, int T,
                               int H, float eps, bool zero_centred, int post_w_stride, int w_stride, cudaStream_t stream);
+void norm_add_f32(float* x, const void* src, bool src_bf16, const int* ids, int rows, const void* w, void* out, bool w_bf16, int T, int H, float eps,
+                  bool zero_centred, cudaStream_t stream);
 void parallel_add_rmsnorm_f32(float* residual, const void* d1, const void* d2, bool delta_bf16, const float* d3, const void* w1, const void* w2, void* out1,
                               void* out2, bool out_bf16, int T, int H, float eps, bool zero_centred, cudaStream_t stream);
 void grouped_rmsnorm(const float* x, const void* w, void* out, bool out_bf16, int T, int C, int groups, float eps, const void* gate, int ldg, int ldo,
@@ -147,10 +153,16 @@ void grouped_rmsnorm(const float* x, const void* w, void* out, bool out_bf16, in
 void bigram_embedding(const void* embed, const void* bigram, bool bf16, const int* ids, int* prev_tokens, const int* cu_q, const int* req_slots,
                       const int* seq_lens, int B, int max_q_len, int W, int vocab, float scale, long long mul_prev, long long mul_cur, int buckets,
                       float* out, cudaStream_t stream);
+void moe_sigmoid_route(const float* logits, int ld, int T, int E, int K, bool renorm, float scale, float* w, int* ids, cudaStream_t stream);
 void moe_softmax_bias_route(const float* logits, int ld, const float* corr, int T, int E, int K, int n_real, float* w, int* ids, float* ident,
                             cudaStream_t stream);
 void moe_identity_shared_combine(void* y, const void* h, const float* ident, const void* shared, const float* gate, bool bf16, int T, int W,
                                  cudaStream_t stream);
+// conv_attention.cu
+void conv_attention_prepare(const void* qkv, int ld, bool bf16, int T, int H, int G, int M, int D, int Dv, const void* conv_w, int taps, void* conv_state,
+                            const int* positions, const int* cu_q, const int* req_slots, const int* seq_lens, int B, const void* q_norm_w,
+                            const void* k_norm_w, float eps, const float* inv_freq, int half, float rot_mult, void* kc, void* vc, size_t ldc,
+                            const int* loc, void* q_out, int pad, int num_sms, cudaStream_t stream);
 // latent_attention.cu
 void latent_attention(const float* q, const void* cache, bool cache_bf16, int ldc, int R, const int* page_table, int pt_stride, int page_size,
                       const int* req_slots, const int* seq_lens, const int* cu_q, int B, int max_q_len, int max_kv_len, int H, float scale,

@@ -45,6 +45,8 @@ constexpr int DA_P_BYTES = 2 * DA_NQ * 128;              // 4 KB   (two 64-key c
 constexpr int DA_SMEM_BYTES = 2 * DA_STAGES * DA_TILE_BYTES + 2 * DA_Q_BYTES + 2 * DA_P_BYTES + 1024 /*align*/ + 1024 /*barriers + scratch*/;
 constexpr float DA_RESCALE_THRESHOLD = 8.0f;
 
+constexpr int DA_PLAIN = 0, DA_CAP = 1, DA_DIFF = 2;      // MODE of a kernel instance
+
 struct DecodeParams {
   __nv_bfloat16* out;     // [B, Hq, D]
   float* part_o;          // [splits, B, Hq, D]
@@ -58,16 +60,19 @@ struct DecodeParams {
   const float* slopes;      // optional [Hq]: distance bias, score -= slopes[h] * (seq_len - 1 - key position), applied after the cap
   const float* log_rates;   // optional [Hq], with slopes: the bias is slopes[h] * ln(1 + log_rates[h] * distance) instead of linear (no cap)
   int window;
+  int chunk;                // > 0: only keys of the query's own chunk of this many positions
+  DiffCombine diff;         // DIFF instances: query heads 2h, 2h + 1 are combined in the epilogue (see attention_tc.cu)
   int keep_first;           // with a window: keys below this position stay visible (their tiles are walked first)
   int total_items;
   int* sched;             // [0] next item, [1] CTAs finished (the last one re-arms both)
   long long* prof;        // PROF builds: [ctas][32] per-role cycle accounting (tools/attn_decode_bench.py prof)
 };
 
-template <int GMAX, bool HAS_CAP, bool PROF>
+template <int GMAX, int MODE, bool PROF>
 __global__ void __launch_bounds__(DA_THREADS, 1)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                    const DecodeParams p) {
+  constexpr bool HAS_CAP = MODE == DA_CAP, DIFF = MODE == DA_DIFF;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int G = p.G;
   extern __shared__ uint8_t smem_raw[];
@@ -147,6 +152,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     it.kv_hi = it.seq_len;
     int kv_lo = 0;
     if (p.window > 0) kv_lo = max(0, it.seq_len - p.window);
+    if (p.chunk > 0) kv_lo = (it.seq_len - 1) / p.chunk * p.chunk;
     const int tile_lo = kv_lo / DA_KT;
     it.keep_tiles = min((p.keep_first + DA_KT - 1) / DA_KT, tile_lo);
     it.tile_skip = tile_lo - it.keep_tiles;
@@ -299,7 +305,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       }
       const int n_tiles = it.n_tiles;
       if (lane == 0) DA_DBG(3, n_q, g);
-      const int kv_first = p.window > 0 ? it.seq_len - p.window : 0;
+      const int kv_first = p.chunk > 0 ? (it.seq_len - 1) / p.chunk * p.chunk : p.window > 0 ? it.seq_len - p.window : 0;
       float slope[GMAX];
 #pragma unroll
       for (int i = 0; i < GMAX; ++i) slope[i] = (HAS_CAP && p.slopes && i < G) ? p.slopes[it.kvh * G + i] : 0.f;
@@ -434,9 +440,31 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(o_free);        // O^T sits in registers: the next item may overwrite the accumulator
+      if (DIFF && p.num_splits == 1) {
+        // pairs of columns: combine, mean square over the output dims (= the 128 threads; red's row-max buffers are idle here), scale, store
+        constexpr int NP = GMAX / 2;
+        float ov[NP];
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const float l0 = sbuf[2 * i] + sbuf[GMAX + 2 * i] + sbuf[2 * GMAX + 2 * i] + sbuf[3 * GMAX + 2 * i];
+          const float l1 = sbuf[2 * i + 1] + sbuf[GMAX + 2 * i + 1] + sbuf[2 * GMAX + 2 * i + 1] + sbuf[3 * GMAX + 2 * i + 1];
+          const float a = l0 > 0.f ? __uint_as_float(orow[2 * i]) / l0 : 0.f, c = l1 > 0.f ? __uint_as_float(orow[2 * i + 1]) / l1 : 0.f;
+          ov[i] = a - p.diff.lam * c;
+          const float ss = warp_sum(ov[i] * ov[i]);
+          if (lane == 0) red[q4 * NP + i] = ss;
+        }
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const float ss = red[i] + red[NP + i] + red[2 * NP + i] + red[3 * NP + i];
+          if (2 * i < G && row < p.diff.dv)
+            p.out[((size_t)it.b * (p.Hq >> 1) + ((it.kvh * G) >> 1) + i) * p.diff.dv + row] =
+                __float2bfloat16(ov[i] * (p.diff.post / sqrtf(ss / (float)p.diff.dv + p.diff.eps)));
+        }
+      }
 #pragma unroll
       for (int i = 0; i < GMAX; ++i) {
-        if (i < G) {
+        if (i < G && !(DIFF && p.num_splits == 1)) {
           const float l = sbuf[i] + sbuf[GMAX + i] + sbuf[2 * GMAX + i] + sbuf[3 * GMAX + i];
           const float inv_l = l > 0.f ? 1.f / l : 0.f;
           const float o = __uint_as_float(orow[i]) * inv_l;
@@ -476,8 +504,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 }
 
 // defined in attention_tc.cu
-__global__ void attn_merge_splits_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, __nv_bfloat16* __restrict__ out,
-                                         float* __restrict__ lse_out, int rows, int num_splits);
+void attn_merge_splits(const float* part_o, const float* part_lse, void* out, float* lse, int rows, int num_splits, const DiffCombine* diff, cudaStream_t stream);
 
 bool attn_decode_tc_supported(int Hq, int Hkv, int D, int page_size) {
   if (D != DA_D || Hkv <= 0 || Hq % Hkv) return false;
@@ -491,7 +518,8 @@ void attn_decode_set_prof(long long* buf) { g_da_prof = buf; }
 void attn_decode_tc(const void* q, const void* k_cache, const void* v_cache, void* out, float* lse, float* part_o, float* part_lse,
                     const int* page_table, int pt_stride, const int* req_slots, const int* seq_lens, int B, int q_stride, int Hq, int Hkv,
                     int D, int num_slots, int page_size, int num_splits, float scale, int window, float logit_cap, int* sched, int num_sms,
-                    cudaStream_t stream, const float* slopes, const float* log_rates, int keep_first, int kv_stride) {
+                    cudaStream_t stream, const float* slopes, const float* log_rates, int keep_first, int kv_stride, int chunk,
+                    const DiffCombine* diff) {
   if (!attn_decode_tc_supported(Hq, Hkv, D, page_size)) throw std::runtime_error("sglb attn_decode_tc: unsupported shape");
   if (sched == nullptr) throw std::runtime_error("sglb attn_decode_tc: needs the work-queue counters");
   const int G = Hq / Hkv;
@@ -514,6 +542,11 @@ void attn_decode_tc(const void* q, const void* k_cache, const void* v_cache, voi
   p.scale_log2 = scale * 1.4426950408889634f; p.logit_cap = logit_cap; p.window = window; p.slopes = slopes;
   p.log_rates = slopes ? log_rates : nullptr; p.keep_first = window > 0 ? std::max(keep_first, 0) : 0;
   if (p.log_rates && logit_cap > 0.f) throw std::runtime_error("sglb attn_decode_tc: the logarithmic distance bias takes no soft cap");
+  p.chunk = chunk > 0 ? chunk : 0;
+  if (p.chunk && window > 0) throw std::runtime_error("sglb attn_decode_tc: chunked attention has no window");
+  p.diff = diff ? *diff : DiffCombine{};
+  if (diff && (G % 2 || lse || logit_cap > 0.f || slopes || diff->dv < 1 || diff->dv > DA_D))
+    throw std::runtime_error("sglb attn_decode_tc: the differential form pairs query heads of a group, without cap, bias or lse; at most 128 value columns");
   p.total_items = B * Hkv * num_splits; p.sched = sched; p.prof = g_da_prof;
   const int ctas = std::min(p.total_items, num_sms);
   const bool capped = logit_cap > 0.f || slopes != nullptr;
@@ -526,24 +559,20 @@ void attn_decode_tc(const void* q, const void* k_cache, const void* v_cache, voi
     }                                                                                                                               \
     attn_decode_kernel<GM_, CAP_, false><<<ctas, DA_THREADS, DA_SMEM_BYTES, stream>>>(tmQ, tmK, tmV, p);                            \
   } while (0)
-  if (g_da_prof != nullptr && G <= 4 && !capped) {      // instrumented build (per-role cycle accounting), bench tool only
+  if (g_da_prof != nullptr && G <= 4 && !capped && !diff) {      // instrumented build (per-role cycle accounting), bench tool only
     static bool configured = false;
     if (!configured) {
-      SGLB_CUDA_CHECK(cudaFuncSetAttribute(attn_decode_kernel<4, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DA_SMEM_BYTES));
+      SGLB_CUDA_CHECK(cudaFuncSetAttribute(attn_decode_kernel<4, DA_PLAIN, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DA_SMEM_BYTES));
       configured = true;
     }
-    attn_decode_kernel<4, false, true><<<ctas, DA_THREADS, DA_SMEM_BYTES, stream>>>(tmQ, tmK, tmV, p);
+    attn_decode_kernel<4, DA_PLAIN, true><<<ctas, DA_THREADS, DA_SMEM_BYTES, stream>>>(tmQ, tmK, tmV, p);
   } else
-  if (G <= 4) { if (capped) SGLB_DA_LAUNCH(4, true); else SGLB_DA_LAUNCH(4, false); }
-  else if (G <= 8) { if (capped) SGLB_DA_LAUNCH(8, true); else SGLB_DA_LAUNCH(8, false); }
-  else { if (capped) SGLB_DA_LAUNCH(16, true); else SGLB_DA_LAUNCH(16, false); }
+  if (G <= 4) { if (diff) SGLB_DA_LAUNCH(4, DA_DIFF); else if (capped) SGLB_DA_LAUNCH(4, DA_CAP); else SGLB_DA_LAUNCH(4, DA_PLAIN); }
+  else if (G <= 8) { if (diff) SGLB_DA_LAUNCH(8, DA_DIFF); else if (capped) SGLB_DA_LAUNCH(8, DA_CAP); else SGLB_DA_LAUNCH(8, DA_PLAIN); }
+  else { if (diff) SGLB_DA_LAUNCH(16, DA_DIFF); else if (capped) SGLB_DA_LAUNCH(16, DA_CAP); else SGLB_DA_LAUNCH(16, DA_PLAIN); }
 #undef SGLB_DA_LAUNCH
   SGLB_CUDA_CHECK(cudaGetLastError());
-  if (num_splits > 1) {
-    const int rows = B * Hq;
-    attn_merge_splits_kernel<<<(rows + 7) / 8, 256, 0, stream>>>(part_o, part_lse, (__nv_bfloat16*)out, lse, rows, num_splits);
-    SGLB_CUDA_CHECK(cudaGetLastError());
-  }
+  if (num_splits > 1) attn_merge_splits(part_o, part_lse, out, lse, B * Hq, num_splits, diff, stream);
 }
 
 }  // namespace sglb

@@ -37,6 +37,10 @@ constexpr int ATT_HALF_BYTES = ATT_TILE_BYTES / 2;
 template <int KT> constexpr int att_smem_bytes() { return ATT_TILE_BYTES + 4 * KT * ATT_D * 2 + 1024 + 256; }
 constexpr float ATT_RESCALE_THRESHOLD = 8.0f;  // log2 units; lazy rescale (FA4-style)
 
+// MODE of a kernel instance: 0 plain, 1 score cap and / or distance bias, 2 differential (neighbouring query heads 2h, 2h + 1 are the two maps of
+// head h: out_h = unit_rms(o_2h - lam * o_2h+1) * post over its first dv columns, [T, Hq / 2, dv])
+constexpr int ATT_PLAIN = 0, ATT_CAP = 1, ATT_DIFF = 2;
+
 struct AttnParams {
   __nv_bfloat16* out;
   float* part_o;      // [splits, T, Hq, D]
@@ -55,13 +59,64 @@ struct AttnParams {
   const float* slopes;        // optional [Hq]: distance bias, score -= slopes[h] * (query position - key position), applied after the cap
   const float* log_rates;     // optional [Hq], with slopes: the bias is slopes[h] * ln(1 + log_rates[h] * distance) instead of linear (no cap)
   int keep_first;             // with a window: keys below this position stay visible to every later query (their tiles are walked first)
+  int chunk;                  // > 0: a query sees only keys of its own chunk of this many positions (counted from position 0 of the sequence)
+  DiffCombine diff;           // DIFF instances: pairs of query heads are combined in the epilogue
   const unsigned* tree_anc;   // speculative tree verify: [T] bit k of tree_anc[t] = query token t may see draft key `prefix + k` (classic launch)
 };
 
-template <int KT, bool HAS_CAP>
+// the two maps of a head sit in neighbouring rows (TMEM lanes) of the tile: every lane forms its pair's combination, sums its square over the
+// row, and writes one half of the columns.  ``o_addr``: the row block of O in TMEM; ``parity``: 0 = map 1, 1 = map 2.
+__device__ __forceinline__ void diff_epilogue(uint32_t o_addr, float inv_l, int parity, bool row_valid, const DiffCombine& d, __nv_bfloat16* dst) {
+  const float coef = parity ? -d.lam * inv_l : inv_l;
+  float ss = 0.f;
+#pragma unroll 1
+  for (int c = 0; c < 4; ++c) {
+    uint32_t orow[32];
+    tmem_ld_32x32b_x32(o_addr + c * 32, orow);
+    tmem_ld_wait();
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      float v = __uint_as_float(orow[i]) * coef;
+      v += __shfl_xor_sync(0xffffffffu, v, 1);
+      ss += v * v;                                   // columns >= dv hold zeros
+    }
+  }
+  const float mul = d.post / sqrtf(ss / (float)d.dv + d.eps);
+  const bool vec = (d.dv & 7) == 0;
+#pragma unroll 1
+  for (int c = 0; c < 4; ++c) {
+    uint32_t orow[32];
+    tmem_ld_32x32b_x32(o_addr + c * 32, orow);
+    tmem_ld_wait();
+    float f[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      float v = __uint_as_float(orow[i]) * coef;
+      v += __shfl_xor_sync(0xffffffffu, v, 1);
+      f[i] = v * mul;
+    }
+    if (!row_valid || (c & 1) != parity) continue;
+    if (vec) {
+#pragma unroll
+      for (int v = 0; v < 4; ++v) {
+        const int col = c * 32 + v * 8;
+        if (col < d.dv)
+          st128(dst + col, U4{pack_bf16(f[v * 8], f[v * 8 + 1]), pack_bf16(f[v * 8 + 2], f[v * 8 + 3]), pack_bf16(f[v * 8 + 4], f[v * 8 + 5]),
+                              pack_bf16(f[v * 8 + 6], f[v * 8 + 7])});
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (c * 32 + i < d.dv) dst[c * 32 + i] = __float2bfloat16(f[i]);
+    }
+  }
+}
+
+template <int KT, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, (KT <= 64) ? 2 : 1)
 attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const AttnParams p) {
+  constexpr bool HAS_CAP = MODE == ATT_CAP, DIFF = MODE == ATT_DIFF;
   const int b = blockIdx.z;
   const int kvh = blockIdx.y / p.num_splits;
   const int split = blockIdx.y % p.num_splits;
@@ -77,6 +132,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   const int kv_hi = p.causal ? min(seq_len, prefix + t_hi) : seq_len;
   int kv_lo = 0;
   if (p.window > 0) kv_lo = max(0, prefix + t0 - p.window + 1);
+  if (p.chunk > 0) kv_lo = (prefix + t0) / p.chunk * p.chunk;
   constexpr int KV_TILE_BYTES = KT * ATT_D * 2;      // K or V tile
   constexpr int KV_HALF_BYTES = KV_TILE_BYTES / 2;   // one 64-wide d-block of the tile
   constexpr int TMEM_COLS = (KT <= 64) ? 256 : 512;  // S0 | S1 | O(128)
@@ -237,7 +293,8 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const float rate = (HAS_CAP && p.log_rates) ? p.log_rates[kvh * G + (r % G)] : 0.f;
     const float log_coef = slope * 0.6931471805599453f * inv_scale_nat;                 // ln(x) = ln 2 * lg2(x), in units of the raw score
     const int kv_last = p.causal ? min(seq_len - 1, q_pos) : seq_len - 1;
-    const int kv_first = p.window > 0 ? q_pos - p.window + 1 : -(1 << 30);
+    const int chunk_edge = p.chunk > 0 ? (prefix + t_hi - 1) / p.chunk * p.chunk : 0;      // first key of the tile's last query's chunk
+    const int kv_first = p.chunk > 0 ? q_pos / p.chunk * p.chunk : p.window > 0 ? q_pos - p.window + 1 : -(1 << 30);
 
     for (int j = 0; j < n_tiles; ++j) {
       const int st = j & 1;
@@ -254,7 +311,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const int Lj = tile_begin + j;
         const int kv0 = (Lj < keep_tiles ? Lj : Lj + tile_skip) * KT;
         const bool need_mask = (kv0 + KT > kv_hi) || (p.causal && kv0 + KT - 1 > prefix + t0) ||
-                               (p.window > 0 && kv0 < prefix + t_hi - p.window);
+                               (p.window > 0 && kv0 < prefix + t_hi - p.window) || kv0 < chunk_edge;
         // The inner loops are kept branch-free and tiny (the 128-wide body is fully unrolled: any per-element branch or
         // constant-bank reload multiplies into thousands of instructions and thrashes the instruction cache).
         if (HAS_CAP && p.log_rates) {   // logarithmic distance bias: raw -= slope * ln(1 + rate * distance) / scale (one FFMA + MUFU.LG2 + FFMA more)
@@ -374,8 +431,11 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       const float lse = (l_i > 0.f) ? (m_i + log2f(l_i)) * 0.6931471805599453f : -INFINITY;
       const int g = r % G;
       const size_t out_row = ((size_t)(q_start + tok)) * p.Hq + kvh * G + g;
+      if constexpr (DIFF) {
+        if (p.num_splits == 1) diff_epilogue(tmem_O + lane_addr, inv_l, r & 1, row_valid, p.diff, p.out + (out_row >> 1) * p.diff.dv);
+      }
 #pragma unroll 1
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < (DIFF && p.num_splits == 1 ? 0 : 4); ++c) {
         uint32_t orow[32];
         tmem_ld_32x32b_x32(tmem_O + lane_addr + c * 32, orow);
         tmem_ld_wait();
@@ -424,10 +484,11 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 // already streaming the next item's Q/K/V while the softmax warps normalise and store the previous one; TMEM, barriers and
 // tensor maps are set up once.  Extra barriers: item ring (item_full/item_empty), q_empty (Q buffer reuse), o_free (O
 // accumulator reuse).  All ring barriers use running counters so phases carry across items.
-template <int KT, bool HAS_CAP>
+template <int KT, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, (KT <= 64) ? 2 : 1)
 attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                            const __grid_constant__ CUtensorMap tmV, const AttnParams p) {
+  constexpr bool HAS_CAP = MODE == ATT_CAP, DIFF = MODE == ATT_DIFF;
   const int G = p.G;
   const int TQ = 128 / G;
   constexpr int KV_TILE_BYTES = KT * ATT_D * 2;
@@ -505,6 +566,7 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     it.kv_hi = p.causal ? min(it.seq_len, it.prefix + it.t_hi) : it.seq_len;
     int kv_lo = 0;
     if (p.window > 0) kv_lo = max(0, it.prefix + it.t0 - p.window + 1);
+    if (p.chunk > 0) kv_lo = (it.prefix + it.t0) / p.chunk * p.chunk;
     const int tile_lo_w = kv_lo / KT;
     it.keep_tiles = min((p.keep_first + KT - 1) / KT, tile_lo_w);
     it.tile_skip = tile_lo_w - it.keep_tiles;
@@ -657,7 +719,8 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       const float log_coef = slope * 0.6931471805599453f * inv_scale_nat;
       float m_i = -INFINITY, l_i = 0.f;
       const int kv_last = p.causal ? min(it.seq_len - 1, q_pos) : it.seq_len - 1;
-      const int kv_first = p.window > 0 ? q_pos - p.window + 1 : -(1 << 30);
+      const int chunk_edge = p.chunk > 0 ? (it.prefix + it.t_hi - 1) / p.chunk * p.chunk : 0;
+      const int kv_first = p.chunk > 0 ? q_pos / p.chunk * p.chunk : p.window > 0 ? q_pos - p.window + 1 : -(1 << 30);
       for (int j = 0; j < n_tiles; ++j) {
         const uint32_t gt = g + j;
         const int st = gt & 1;
@@ -673,7 +736,7 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           tmem_ld_wait();
           const int kv0 = it.tile(j) * KT;
           const bool need_mask = (kv0 + KT > it.kv_hi) || (p.causal && kv0 + KT - 1 > it.prefix + it.t0) ||
-                                 (p.window > 0 && kv0 < it.prefix + it.t_hi - p.window);
+                                 (p.window > 0 && kv0 < it.prefix + it.t_hi - p.window) || kv0 < chunk_edge;
           if (HAS_CAP && p.log_rates) {
             const float d0 = (float)(q_pos - kv0);
 #pragma unroll
@@ -774,8 +837,11 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         const float lse = (l_i > 0.f) ? (m_i + log2f(l_i)) * 0.6931471805599453f : -INFINITY;
         const int gq = r % G;
         const size_t out_row = ((size_t)(it.q_start + tok)) * p.Hq + it.kvh * G + gq;
+        if constexpr (DIFF) {
+          if (p.num_splits == 1) diff_epilogue(tmem_O + lane_addr, inv_l, r & 1, row_valid, p.diff, p.out + (out_row >> 1) * p.diff.dv);
+        }
 #pragma unroll 1
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < (DIFF && p.num_splits == 1 ? 0 : 4); ++c) {
           uint32_t orow[32];
           tmem_ld_32x32b_x32(tmem_O + lane_addr + c * 32, orow);
           tmem_ld_wait();
@@ -854,11 +920,54 @@ __global__ void attn_merge_splits_kernel(const float* __restrict__ part_o, const
   if (lse_out && lane == 0) lse_out[row] = wsum > 0.f ? m + __logf(wsum) : -INFINITY;
 }
 
+// the same for the differential form: one warp per (token, pair of query heads)
+__global__ void attn_merge_splits_diff_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, __nv_bfloat16* __restrict__ out,
+                                              int pairs, int num_splits, const DiffCombine d) {
+  const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (pair >= pairs) return;
+  const size_t rows = (size_t)2 * pairs;
+  float o[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int mp = 0; mp < 2; ++mp) {
+    const size_t row = (size_t)2 * pair + mp;
+    float m = -INFINITY;
+    for (int s = 0; s < num_splits; ++s) m = fmaxf(m, part_lse[(size_t)s * rows + row]);
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    float wsum = 0.f;
+    for (int s = 0; s < num_splits; ++s) {
+      const float l = part_lse[(size_t)s * rows + row];
+      const float w = (l == -INFINITY) ? 0.f : __expf(l - m);
+      wsum += w;
+      const float4 v = *reinterpret_cast<const float4*>(part_o + ((size_t)s * rows + row) * ATT_D + lane * 4);
+      acc[0] += w * v.x; acc[1] += w * v.y; acc[2] += w * v.z; acc[3] += w * v.w;
+    }
+    const float f = (wsum > 0.f ? 1.f / wsum : 0.f) * (mp ? -d.lam : 1.f);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) o[i] += acc[i] * f;
+  }
+  const float ss = warp_sum(o[0] * o[0] + o[1] * o[1] + o[2] * o[2] + o[3] * o[3]);
+  const float mul = d.post / sqrtf(ss / (float)d.dv + d.eps);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (lane * 4 + i < d.dv) out[(size_t)pair * d.dv + lane * 4 + i] = __float2bfloat16(o[i] * mul);
+}
+
+void attn_merge_splits(const float* part_o, const float* part_lse, void* out, float* lse, int rows, int num_splits, const DiffCombine* diff,
+                       cudaStream_t stream) {
+  if (diff) {
+    attn_merge_splits_diff_kernel<<<(rows / 2 + 7) / 8, 256, 0, stream>>>(part_o, part_lse, (__nv_bfloat16*)out, rows / 2, num_splits, *diff);
+  } else {
+    attn_merge_splits_kernel<<<(rows + 7) / 8, 256, 0, stream>>>(part_o, part_lse, (__nv_bfloat16*)out, lse, rows, num_splits);
+  }
+  SGLB_CUDA_CHECK(cudaGetLastError());
+}
+
 void attn_fwd_tc(const void* q, const void* k_cache, const void* v_cache, void* out, float* lse, float* part_o,
                  float* part_lse, const int* page_table, int pt_stride, const int* req_slots, const int* seq_lens,
                  const int* cu_q, int B, int T, int q_stride, int max_q_len, int Hq, int Hkv, int D, int num_slots, int page_size,
                  int num_splits, float scale, int causal, int window, float logit_cap, int* sched, int num_sms,
-                 cudaStream_t stream, const unsigned* tree_anc, const float* slopes, const float* log_rates, int keep_first, int kv_stride) {
+                 cudaStream_t stream, const unsigned* tree_anc, const float* slopes, const float* log_rates, int keep_first, int kv_stride,
+                 int chunk, const DiffCombine* diff) {
   if (D != ATT_D) throw std::runtime_error("sglb attn_tc: head_dim must be 128");
   const int G = Hq / Hkv;
   if (G < 1 || G > 128 || (128 % G) != 0) throw std::runtime_error("sglb attn_tc: GQA group must divide 128");
@@ -883,6 +992,11 @@ void attn_fwd_tc(const void* q, const void* k_cache, const void* v_cache, void* 
   p.scale_log2 = scale * 1.4426950408889634f; p.logit_cap = logit_cap; p.causal = causal; p.window = window;
   p.tree_anc = tree_anc; p.slopes = slopes;
   p.log_rates = slopes ? log_rates : nullptr; p.keep_first = window > 0 ? std::max(keep_first, 0) : 0;
+  p.chunk = chunk > 0 ? chunk : 0;
+  if (p.chunk && (window > 0 || !causal || tree_anc)) throw std::runtime_error("sglb attn_tc: chunked attention is causal, without a window or a tree");
+  p.diff = diff ? *diff : DiffCombine{};
+  if (diff && (G % 2 || lse || logit_cap > 0.f || slopes || diff->dv < 1 || diff->dv > ATT_D))
+    throw std::runtime_error("sglb attn_tc: the differential form pairs query heads of a group, without cap, bias or lse; at most 128 value columns");
   if (p.log_rates && logit_cap > 0.f) throw std::runtime_error("sglb attn_tc: the logarithmic distance bias takes no soft cap");
   if (tree_anc != nullptr) {
     if (max_q_len > 32 || num_splits != 1 || window > 0) throw std::runtime_error("sglb attn_tc: tree masks cover <= 32 draft nodes, no split-KV / window");
@@ -917,20 +1031,16 @@ void attn_fwd_tc(const void* q, const void* k_cache, const void* v_cache, void* 
   // persistent scheduling pays off once there are more items than resident CTAs (otherwise the classic launch is identical)
   const bool persist = sched != nullptr && tree_anc == nullptr && p.total_items > num_sms * (small ? 2 : 1);
   if (persist) {
-    if (small) { if (capped) SGLB_ATT_LAUNCH_P(64, true); else SGLB_ATT_LAUNCH_P(64, false); }
-    else { if (capped) SGLB_ATT_LAUNCH_P(128, true); else SGLB_ATT_LAUNCH_P(128, false); }
+    if (small) { if (diff) SGLB_ATT_LAUNCH_P(64, ATT_DIFF); else if (capped) SGLB_ATT_LAUNCH_P(64, ATT_CAP); else SGLB_ATT_LAUNCH_P(64, ATT_PLAIN); }
+    else { if (diff) SGLB_ATT_LAUNCH_P(128, ATT_DIFF); else if (capped) SGLB_ATT_LAUNCH_P(128, ATT_CAP); else SGLB_ATT_LAUNCH_P(128, ATT_PLAIN); }
   } else {
-    if (small) { if (capped) SGLB_ATT_LAUNCH(64, true); else SGLB_ATT_LAUNCH(64, false); }
-    else { if (capped) SGLB_ATT_LAUNCH(128, true); else SGLB_ATT_LAUNCH(128, false); }
+    if (small) { if (diff) SGLB_ATT_LAUNCH(64, ATT_DIFF); else if (capped) SGLB_ATT_LAUNCH(64, ATT_CAP); else SGLB_ATT_LAUNCH(64, ATT_PLAIN); }
+    else { if (diff) SGLB_ATT_LAUNCH(128, ATT_DIFF); else if (capped) SGLB_ATT_LAUNCH(128, ATT_CAP); else SGLB_ATT_LAUNCH(128, ATT_PLAIN); }
   }
 #undef SGLB_ATT_LAUNCH
 #undef SGLB_ATT_LAUNCH_P
   SGLB_CUDA_CHECK(cudaGetLastError());
-  if (num_splits > 1) {
-    const int rows = T * Hq;
-    attn_merge_splits_kernel<<<(rows + 7) / 8, 256, 0, stream>>>(part_o, part_lse, (__nv_bfloat16*)out, lse, rows, num_splits);
-    SGLB_CUDA_CHECK(cudaGetLastError());
-  }
+  if (num_splits > 1) attn_merge_splits(part_o, part_lse, out, lse, T * Hq, num_splits, diff, stream);
 }
 
 }  // namespace sglb

@@ -16,6 +16,8 @@
 #include <stdint.h>
 #include <stdio.h>
 
+#include "params.h"
+
 namespace sglb {
 
 // ---------------------------------------------------------------- misc

@@ -19,10 +19,11 @@ constexpr int GEMM_BM = 128;
 constexpr int GEMM_BK = 64;
 constexpr int GEMM_THREADS = 256;
 
-enum GemmEpilogue { EPI_NONE = 0, EPI_BIAS = 1, EPI_SILU_MUL = 2, EPI_PUSH = 3, EPI_SILU_SPLIT = 4, EPI_ROWSCALE = 5 };
+enum GemmEpilogue { EPI_NONE = 0, EPI_BIAS = 1, EPI_SILU_MUL = 2, EPI_PUSH = 3, EPI_SILU_SPLIT = 4, EPI_ROWSCALE = 5, EPI_RELU2 = 6 };
 // EPI_SILU_SPLIT: W = [gate rows (n_half) ; up rows (n_half)] un-interleaved (the checkpoint layout).  Each B stage is
 //   filled by TWO TMA boxes of BN/2 rows — gate rows j.. and up rows n_half+j.. — so one UMMA of width BN produces the
 //   gate half in accumulator columns [0,BN/2) and the matching up half in [BN/2,BN); the epilogue writes silu(g)*u.
+// EPI_RELU2    : C = max(acc, 0)^2 (ungated experts).
 // EPI_ROWSCALE : C[row,:] = acc[row,:] * scale[row]  (fp32 per-row scale passed through `bias`; MoE routing weights).
 // GROUPED      : A rows are expert-sorted and padded to 128-row tiles; W is [E][N][K] behind a 3-D tensor map and
 //   tile_expert[m_tile] selects the expert slab; the number of live M tiles is read from device memory.
@@ -210,6 +211,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
 #pragma unroll
                   for (int i = 0; i < 8; ++i) f[i] *= row_scale;
                 }
+                if (EPI == EPI_RELU2) {
+#pragma unroll
+                  for (int i = 0; i < 8; ++i) { const float a = fmaxf(f[i], 0.f); f[i] = a * a; }
+                }
                 if (EPI == EPI_BIAS) {
                   U4 b = ldg128(bias + col);
                   f[0] += bf16_lo(b.x); f[1] += bf16_hi(b.x); f[2] += bf16_lo(b.y); f[3] += bf16_hi(b.y);
@@ -360,10 +365,11 @@ void gemm_bf16_tc(const void* A, const void* W, void* C, const void* bias, int M
 
 // Expert-grouped GEMM over expert-sorted, 128-row-padded activations (see moe.cu for the alignment kernels).
 //   split_silu: W = [E][2*n_out][K] (gate;up), C = [M_cap][n_out] = silu(gate)*up
+//   relu2      : W = [E][n_out][K],             C = [M_cap][n_out] = max(acc, 0)^2
 //   else      : W = [E][n_out][K],             C = [M_cap][n_out] = acc * row_scale[row]   (row_scale may be null)
 void gemm_bf16_tc_grouped(const void* A, const void* W, void* C, const float* row_scale, int M_cap, int n_out, int K, int lda,
                           int ldc, int num_experts, const int* tile_expert, const int* num_m_tiles, bool split_silu, int num_sms,
-                          cudaStream_t stream) {
+                          cudaStream_t stream, bool relu2) {
   if (M_cap <= 0 || n_out <= 0) return;
   if (K % 8 || n_out % 32 || lda % 8) throw std::runtime_error("sglb grouped gemm: K % 8, n_out % 32, lda % 8 required");
   GemmExtra ex; ex.num_experts = num_experts; ex.tile_expert = tile_expert; ex.num_m_tiles = num_m_tiles;
@@ -386,7 +392,8 @@ void gemm_bf16_tc_grouped(const void* A, const void* W, void* C, const float* ro
       if ((long long)m_tiles * (n_out / cand) >= 2LL * num_sms) break;
     }
     if (!bn) throw std::runtime_error("sglb grouped gemm: n_out must be a multiple of 32");
-    if (row_scale) dispatch_bn<EPI_ROWSCALE, true>(bn, A, W, C, row_scale, M_cap, n_out, K, lda, K, ldc, num_sms, stream, GemmPush{}, ex);
+    if (relu2) dispatch_bn<EPI_RELU2, true>(bn, A, W, C, nullptr, M_cap, n_out, K, lda, K, ldc, num_sms, stream, GemmPush{}, ex);
+    else if (row_scale) dispatch_bn<EPI_ROWSCALE, true>(bn, A, W, C, row_scale, M_cap, n_out, K, lda, K, ldc, num_sms, stream, GemmPush{}, ex);
     else dispatch_bn<EPI_NONE, true>(bn, A, W, C, nullptr, M_cap, n_out, K, lda, K, ldc, num_sms, stream, GemmPush{}, ex);
   }
 }

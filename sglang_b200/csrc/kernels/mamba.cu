@@ -107,6 +107,36 @@ __global__ void __launch_bounds__(256) causal_conv1d_state_kernel(const T* __res
     if (j < K - 1) st_f<T>(st + j, nw[j]);
 }
 
+// the state half alone, for kernels that convolve on their own (any number of taps: columns are moved one by one, oldest first)
+template <typename T>
+__global__ void __launch_bounds__(256) conv_state_roll_kernel(const T* __restrict__ x, int ldx, T* __restrict__ conv_state, const int* __restrict__ cu_q,
+                                                              const int* __restrict__ req_slots, const int* __restrict__ seq_lens, int C, int K) {
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  const int b = blockIdx.y;
+  if (c >= C) return;
+  const int q0 = cu_q ? cu_q[b] : b;
+  const int n = cu_q ? cu_q[b + 1] - q0 : 1;
+  if (n <= 0) return;
+  const bool fresh = seq_lens[b] - n == 0;
+  T* st = conv_state + ((size_t)req_slots[b] * C + c) * (K - 1);
+  for (int j = 0; j < K - 1; ++j) {                  // column j takes input n - (K - 1) + j; an old input comes from column j + n > j, not yet overwritten
+    const int t = n - (K - 1) + j;
+    st[j] = t >= 0 ? x[(size_t)(q0 + t) * ldx + c] : fresh ? (T)0.f : st[j + n];
+  }
+}
+
+void causal_conv1d_state(const void* x, int ldx, void* conv_state, const int* cu_q, const int* req_slots, const int* seq_lens, int B, int C, int K,
+                         bool bf16, cudaStream_t stream) {
+  if (B <= 0 || K < 2) return;
+  if (B > 65535) throw std::runtime_error("sglb causal_conv1d_state: at most 65535 requests");
+  dim3 grid((C + 255) / 256, B);
+  if (bf16)
+    conv_state_roll_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)conv_state, cu_q, req_slots, seq_lens, C, K);
+  else
+    conv_state_roll_kernel<float><<<grid, 256, 0, stream>>>((const float*)x, ldx, (float*)conv_state, cu_q, req_slots, seq_lens, C, K);
+  SGLB_CUDA_CHECK(cudaGetLastError());
+}
+
 void causal_conv1d(const void* x, int ldx, const void* w, const void* bias, void* conv_state, const int* cu_q, const int* req_slots,
                    const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, float* u, int ldu, cudaStream_t stream) {
   if (B <= 0) return;

@@ -6,7 +6,8 @@
 //                      (the GEMM's M tile), producing sorted_row[pos] -> pair, inv_pos[pair] -> pos, the per-row
 //                      routing weight, tile_expert[m_tile] and the number of live M tiles — all in device memory, so
 //                      the whole MoE block is CUDA-graph capturable with no host round trip.
-//   moe_gather         xs[pos,:] = x[sorted_row[pos] / K, :]     (zeros for padding rows)
+//   moe_gather         xs[pos,:] = x[sorted_row[pos] / K, :]     (zeros for padding rows), optionally times the pair's routing weight (routers
+//                      whose weight multiplies an expert's input)
 //   moe_combine        out[t,:] = sum_k ys[inv_pos[t*K+k],:]     (fixed k order -> deterministic), optionally PUSHED into
 //                      slot [rank] of every peer's NVLink arena so the expert-parallel all-reduce needs no further kernel
 //                      on the producer side (consumer: nvl_local_reduce_add_rmsnorm in comm/nvl_allreduce.cu).
@@ -149,9 +150,10 @@ void moe_align(const int* topk_ids, const float* topk_w, int n_pairs, int E, int
 }
 
 // ---------------------------------------------------------------- gather into expert-sorted order
+template <bool SCALE>
 __global__ void __launch_bounds__(256) moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ sorted_row,
                                                          const int* __restrict__ num_tiles, __nv_bfloat16* __restrict__ xs, int H,
-                                                         int x_stride, int K, int cap_rows) {
+                                                         int x_stride, int K, int cap_rows, const float* __restrict__ row_w) {
   const int live = min(cap_rows, __ldg(num_tiles) * MOE_TILE);
   const int nvec = H >> 3;
   for (int row = blockIdx.x; row < live; row += gridDim.x) {
@@ -159,7 +161,16 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const __nv_bfloat16* __
     __nv_bfloat16* dst = xs + (size_t)row * H;
     if (pair >= 0) {
       const __nv_bfloat16* src = x + (size_t)(pair / K) * x_stride;
-      for (int v = threadIdx.x; v < nvec; v += blockDim.x) st128(dst + v * 8, ldg128(src + v * 8));
+      if (SCALE) {
+        const float w = __ldg(row_w + row);
+        for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
+          const U4 a = ldg128(src + v * 8);
+          st128(dst + v * 8, U4{pack_bf16(bf16_lo(a.x) * w, bf16_hi(a.x) * w), pack_bf16(bf16_lo(a.y) * w, bf16_hi(a.y) * w),
+                                pack_bf16(bf16_lo(a.z) * w, bf16_hi(a.z) * w), pack_bf16(bf16_lo(a.w) * w, bf16_hi(a.w) * w)});
+        }
+      } else {
+        for (int v = threadIdx.x; v < nvec; v += blockDim.x) st128(dst + v * 8, ldg128(src + v * 8));
+      }
     } else {
       for (int v = threadIdx.x; v < nvec; v += blockDim.x) st128(dst + v * 8, U4{0, 0, 0, 0});
     }
@@ -167,11 +178,13 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const __nv_bfloat16* __
 }
 
 void moe_gather(const void* x, const int* sorted_row, const int* num_tiles, void* xs, int H, int x_stride, int K, int cap_rows,
-                int num_sms, cudaStream_t stream) {
+                int num_sms, cudaStream_t stream, const float* row_w) {
   if (H % 8) throw std::runtime_error("sglb moe_gather: hidden size must be a multiple of 8");
   const int grid = max(1, min(cap_rows, num_sms * 8));
-  moe_gather_kernel<<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, sorted_row, num_tiles, (__nv_bfloat16*)xs, H, x_stride, K,
-                                              cap_rows);
+  if (row_w)
+    moe_gather_kernel<true><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, sorted_row, num_tiles, (__nv_bfloat16*)xs, H, x_stride, K, cap_rows, row_w);
+  else
+    moe_gather_kernel<false><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, sorted_row, num_tiles, (__nv_bfloat16*)xs, H, x_stride, K, cap_rows, nullptr);
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
 
@@ -314,6 +327,50 @@ void moe_softmax_bias_route(const float* logits, int ld, const float* corr, int 
   if (T <= 0) return;
   if (E > 1024 || K > E) throw std::runtime_error("sglb moe_softmax_bias_route: at most 1024 router columns, top_k <= columns");
   moe_softmax_bias_route_kernel<<<(T + 3) / 4, 128, sizeof(float) * 8 * E, stream>>>(logits, ld, corr, T, E, K, n_real, w, ids, ident);
+  SGLB_CUDA_CHECK(cudaGetLastError());
+}
+
+// ---------------------------------------------------------------- sigmoid router: the K largest logits win and are weighted sigmoid(logit) (times scale;
+// renorm: divided by their sum first).  One warp per token; the choice works on the logits, whose order is that of the scores.
+__global__ void __launch_bounds__(128) moe_sigmoid_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int K, int renorm, float scale,
+                                                                float* __restrict__ w, int* __restrict__ ids) {
+  extern __shared__ float rsm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + warp;
+  if (t >= T) return;
+  float* ch = rsm + (size_t)warp * E;
+  const float* row = logits + (size_t)t * ld;
+  for (int e = lane; e < E; e += 32) ch[e] = row[e];
+  __syncwarp();
+  float mine = 0.f, sum = 0.f;                          // lane k keeps pick k (K <= 32)
+  int my_id = 0;
+  for (int k = 0; k < K; ++k) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32)
+      if (ch[e] > best || bi == 0x7fffffff) { best = ch[e]; bi = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) { best = ob; bi = oi; }
+    }
+    const float sv = 1.f / (1.f + expf(-best));
+    sum += sv;
+    if (lane == k) { mine = sv; my_id = bi; }
+    if (lane == 0) ch[bi] = -INFINITY;
+    __syncwarp();
+  }
+  if (lane < K) {
+    w[(size_t)t * K + lane] = (renorm ? mine / sum : mine) * scale;
+    ids[(size_t)t * K + lane] = my_id;
+  }
+}
+
+void moe_sigmoid_route(const float* logits, int ld, int T, int E, int K, bool renorm, float scale, float* w, int* ids, cudaStream_t stream) {
+  if (T <= 0) return;
+  if (E > 2048 || K > E || K > 32) throw std::runtime_error("sglb moe_sigmoid_route: at most 2048 experts, top_k <= min(32, experts)");
+  moe_sigmoid_route_kernel<<<(T + 3) / 4, 128, sizeof(float) * 4 * E, stream>>>(logits, ld, T, E, K, renorm ? 1 : 0, scale, w, ids);
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
 

@@ -217,6 +217,54 @@ __global__ void __launch_bounds__(256) parallel_add_rmsnorm_f32_kernel(float* __
   }
 }
 
+// x += rmsnorm(src) * (one + w), or x = ... when ``ids`` picks the source row from a table (embedding);  out = x in TO (optional): the residual update
+// of a block that norms a sublayer's output only, so that the next sublayer reads the stream itself.  VEC = 4: four columns per access, up to four
+// accesses of the row in registers.
+template <typename TS, typename TO, int VEC>
+__global__ void __launch_bounds__(256) norm_add_f32_kernel(float* __restrict__ x, const TS* __restrict__ src, const int* __restrict__ ids, int rows,
+                                                           const TO* __restrict__ w, TO* __restrict__ out, int H, float eps, float one) {
+  __shared__ float red[8];
+  const size_t off = (size_t)blockIdx.x * H;
+  const TS* s = ids ? src + (size_t)min(max(ids[blockIdx.x], 0), rows - 1) * H : src + off;
+  float ss = 0.f;
+  if constexpr (VEC == 4) {
+    constexpr int KEEP = 4;
+    float4 keep[KEEP];
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = (threadIdx.x + k * 256) * 4;
+      keep[k] = i < H ? ld4f<TS>(s + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += keep[k].x * keep[k].x + keep[k].y * keep[k].y + keep[k].z * keep[k].z + keep[k].w * keep[k].w;
+    }
+    for (int i = (threadIdx.x + KEEP * 256) * 4; i < H; i += 1024) {          // rows wider than 4096: the rest is read again below
+      const float4 v = ld4f<TS>(s + i);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    const float rs = 1.0f / sqrtf(block_sum_256(ss, red) / (float)H + eps);
+    auto emit = [&](int i, float4 v) {
+      const float4 a = ld4f<TO>(w + i);
+      float4 r = ids ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(x + off + i);
+      r.x += v.x * rs * (one + a.x); r.y += v.y * rs * (one + a.y); r.z += v.z * rs * (one + a.z); r.w += v.w * rs * (one + a.w);
+      *reinterpret_cast<float4*>(x + off + i) = r;
+      if (out) st4f<TO>(out + off + i, r);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = (threadIdx.x + k * 256) * 4;
+      if (i < H) emit(i, keep[k]);
+    }
+    for (int i = (threadIdx.x + KEEP * 256) * 4; i < H; i += 1024) emit(i, ld4f<TS>(s + i));
+  } else {
+    for (int i = threadIdx.x; i < H; i += 256) { const float v = ldf<TS>(s + i); ss += v * v; }
+    const float rs = 1.0f / sqrtf(block_sum_256(ss, red) / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += 256) {
+      const float r = (ids ? 0.f : x[off + i]) + ldf<TS>(s + i) * rs * (one + ldf<TO>(w + i));
+      x[off + i] = r;
+      if (out) stf<TO>(out + off + i, r);
+    }
+  }
+}
+
 // x fp32 [T, C] in ``groups`` equal parts: part / sqrt(mean(part^2) + eps) * w [* sigmoid(gate)] * out_scale; grid (T, groups); gate and out are
 // rows of ldg / ldo elements
 template <typename TO>
@@ -285,6 +333,24 @@ void postnorm_add_rmsnorm_f32(float* residual, const void* delta, bool delta_bf1
       postnorm_add_rmsnorm_f32_kernel<float, float><<<T, 256, 0, stream>>>(residual, (const float*)delta, (const float*)post_w, (const float*)w,
                                                                            (float*)out, H, eps, one, wsp, ws);
   }
+  SGLB_CUDA_CHECK(cudaGetLastError());
+}
+
+void norm_add_f32(float* x, const void* src, bool src_bf16, const int* ids, int rows, const void* w, void* out, bool w_bf16, int T, int H, float eps,
+                  bool zero_centred, cudaStream_t stream) {
+  if (T <= 0) return;
+  using bf = __nv_bfloat16;
+  const float one = zero_centred ? 1.f : 0.f;
+  auto al = [](const void* p) { return p == nullptr || ((uintptr_t)p % 16) == 0; };
+  const bool vec = H % 4 == 0 && al(x) && al(src) && al(w) && al(out);
+#define SGLB_NA(TS, TO)                                                                                                                             \
+  do {                                                                                                                                              \
+    if (vec) norm_add_f32_kernel<TS, TO, 4><<<T, 256, 0, stream>>>(x, (const TS*)src, ids, rows, (const TO*)w, (TO*)out, H, eps, one);                \
+    else norm_add_f32_kernel<TS, TO, 1><<<T, 256, 0, stream>>>(x, (const TS*)src, ids, rows, (const TO*)w, (TO*)out, H, eps, one);                    \
+  } while (0)
+  if (w_bf16) { if (src_bf16) SGLB_NA(bf, bf); else SGLB_NA(float, bf); }
+  else { if (src_bf16) SGLB_NA(bf, float); else SGLB_NA(float, float); }
+#undef SGLB_NA
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
 

@@ -8,6 +8,8 @@
 //                         Options: the sequence's first ``keep_first`` positions stay visible behind the window (their tiles are walked before
 //                         the window's); the bias is slope_h * ln(1 + rate_h * (i - j)) instead of linear; the output is multiplied by
 //                         sigmoid(gate) per head or per element and by a constant in the epilogue, and may be a column block of a wider buffer.
+//                         ``chunk``: a query sees only keys of its own stretch of that many positions (counted from position 0).  Differential form:
+//                         query heads 2h, 2h + 1 are two maps over the same values and are combined in the epilogue (DiffCombine).
 //   attention_prepare   : per token, q and k RMS-normed over their whole projection times a weight, the first coordinates of every head
 //                         rotated by position (pairs half a rotary width apart), v blended with another layer's values, k / v rows to the cache.
 //   sigmoid_gate        : o[:, :, :Dv] * sigmoid(gate) * constant, for attention kernels without a gate epilogue.
@@ -94,6 +96,8 @@ struct WinAttnParams {
   int H, G, HG, HC, nchunks, QT, D, Dp, Dv;
   int Dq, hsk, hsv;                            // head strides of q and of the key / value rows (>= D, D, Dv: padded layouts)
   float scale, softcap; int window;
+  int chunk;                                   // > 0: chunked visibility
+  int is_diff; DiffCombine diff;               // is_diff: out is [T, H / 2, Dv]
   int vec;                                     // 16-byte gathers: head sizes, row stride and base addresses allow them
 };
 
@@ -141,7 +145,7 @@ __global__ void __launch_bounds__(WA_NT) window_attention_kernel(const WinAttnPa
   // ---- per-row constants and online soft-max state (the sink is the first term: max = sink, sum = 1)
   const int r0 = warp * 4;
   float m[4], l[4], slope[4], rate[4], O[4][CV];
-  int qpos[4];
+  int qpos[4], first[4];                                // first[r]: first key of the row's chunk
   bool rowok[4];
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
@@ -149,6 +153,7 @@ __global__ void __launch_bounds__(WA_NT) window_attention_kernel(const WinAttnPa
     rowok[r] = qi < nq && hc < nh;
     const int h = hbase + (rowok[r] ? hc : 0);
     qpos[r] = pos0 + qi;
+    first[r] = p.chunk > 0 ? qpos[r] / p.chunk * p.chunk : 0;
     slope[r] = p.slopes ? p.slopes[h] : 0.f;
     rate[r] = p.log_rates ? p.log_rates[h] : 0.f;
     m[r] = p.sinks ? p.sinks[h] : -INFINITY;
@@ -156,7 +161,7 @@ __global__ void __launch_bounds__(WA_NT) window_attention_kernel(const WinAttnPa
 #pragma unroll
     for (int c = 0; c < CV; ++c) O[r][c] = 0.f;
   }
-  const int klo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  const int klo = p.chunk > 0 ? pos0 / p.chunk * p.chunk : p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int kend = pos0 + nq;                           // one past the last key any query of the tile sees
   const int nkeep = min(p.keep_first, klo);             // kept first positions that lie before the window: a segment of their own
   const int* pt = p.page_table + (size_t)p.req_slots[b] * p.pt_stride;
@@ -238,7 +243,7 @@ __global__ void __launch_bounds__(WA_NT) window_attention_kernel(const WinAttnPa
         if (p.softcap > 0.f) v = p.softcap * tanhf(v * inv_cap);
         if (p.log_rates) v -= slope[r] * log1pf(rate[r] * (float)max(dist, 0));
         else v -= slope[r] * (float)dist;
-        const bool vis = rowok[r] && j < khi && dist >= 0 && (p.window <= 0 || dist < p.window || j < p.keep_first);
+        const bool vis = rowok[r] && j < khi && dist >= 0 && j >= first[r] && (p.window <= 0 || dist < p.window || j < p.keep_first);
         s[kk] = vis ? v : -INFINITY;
       }
       const float mt = warp_max(fmaxf(s[0], s[1]));
@@ -273,6 +278,26 @@ __global__ void __launch_bounds__(WA_NT) window_attention_kernel(const WinAttnPa
   }
   T* og = reinterpret_cast<T*>(p.out);
   const T* gg = reinterpret_cast<const T*>(p.gate);
+  if (p.is_diff) {                                      // rows (0, 1) and (2, 3) of the warp are the map pairs of two heads
+#pragma unroll
+    for (int r = 0; r < 4; r += 2) {
+      if (!rowok[r]) continue;                          // warp-uniform
+      const int qi = (r0 + r) / HC, hc = (r0 + r) - qi * HC;
+      const float f0 = l[r] > 0.f ? 1.f / l[r] : 0.f, f1 = l[r + 1] > 0.f ? p.diff.lam / l[r + 1] : 0.f;
+      float ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < CV; ++c) {
+        O[r][c] = O[r][c] * f0 - O[r + 1][c] * f1;
+        if (lane + 32 * c < Dv) ss += O[r][c] * O[r][c];
+      }
+      const float mul = p.diff.post / sqrtf(warp_sum(ss) / (float)Dv + p.diff.eps);
+      T* dst = og + (size_t)(q0 + qt0 + qi) * p.ldo + (size_t)((hbase + hc) >> 1) * Dv;
+#pragma unroll
+      for (int c = 0; c < CV; ++c)
+        if (lane + 32 * c < Dv) wa_st<T>(dst + lane + 32 * c, O[r][c] * mul);
+    }
+    return;
+  }
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
     if (!rowok[r]) continue;
@@ -703,8 +728,10 @@ void qk_norm_cache_write(const void* qkv, int ld, bool bf16, int T, int H, int G
 void window_attention(const void* q, const void* kc, const void* vc, bool bf16, size_t ldc, int H, int G, int D, int Dv, const int* page_table,
                       int pt_stride, int page_size, const int* req_slots, const int* seq_lens, const int* cu_q, int B, int max_q_len, float scale,
                       float softcap, int window, const float* slopes, const float* sinks, void* out, int pad, int keep_first, const float* log_rates,
-                      const void* gate, int ldg, bool gate_per_head, int ldo, float out_scale, cudaStream_t stream) {
+                      const void* gate, int ldg, bool gate_per_head, int ldo, float out_scale, int chunk, const DiffCombine* diff, cudaStream_t stream) {
   if (B <= 0 || max_q_len <= 0) return;
+  if (chunk > 0 && window > 0) throw std::runtime_error("sglb window_attention: a chunk and a window exclude each other");
+  if (diff && ((H / G) % 2 || gate || out_scale != 1.f)) throw std::runtime_error("sglb window_attention: the differential form pairs the query heads of a group, without a gate");
   if (D > 256 || Dv > 256 || B > 65535 || H % G) throw std::runtime_error("sglb window_attention: head sizes up to 256, heads a multiple of key heads");
   WinAttnParams p;
   p.q = q; p.kc = kc; p.vc = vc; p.out = out; p.ldc = ldc;
@@ -712,6 +739,8 @@ void window_attention(const void* q, const void* kc, const void* vc, bool bf16, 
   p.req_slots = req_slots; p.seq_lens = seq_lens; p.cu_q = cu_q; p.slopes = slopes; p.sinks = sinks;
   p.log_rates = slopes ? log_rates : nullptr; p.gate = gate; p.ldg = ldg; p.gate_per_head = gate_per_head ? 1 : 0; p.ldo = ldo; p.out_scale = out_scale;
   p.keep_first = window > 0 ? std::max(0, keep_first) : 0;
+  p.chunk = chunk > 0 ? chunk : 0;
+  p.is_diff = diff ? 1 : 0; p.diff = diff ? *diff : DiffCombine{};
   p.H = H; p.G = G; p.HG = H / G;
   p.HC = std::min(p.HG, WA_ROWS);
   p.nchunks = (p.HG + p.HC - 1) / p.HC;

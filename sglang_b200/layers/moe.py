@@ -63,7 +63,7 @@ def softmax_bias_route(logits: torch.Tensor, correction, top_k: int, n_real: int
 
 class FusedMoE(nn.Module):
     def __init__(self, num_experts: int, top_k: int, hidden_size: int, intermediate_size: int, dtype=torch.bfloat16,
-                 renormalize: bool = True, ep_size: int = 1, quant=None, layer_id: int = 0):
+                 renormalize: bool = True, ep_size: int = 1, quant=None, layer_id: int = 0, gated: bool = True):
         super().__init__()
         self.tp = get_tp_group()
         self.num_experts, self.top_k, self.renormalize, self.layer_id = num_experts, top_k, renormalize, layer_id
@@ -80,9 +80,11 @@ class FusedMoE(nn.Module):
         self.expert_offset = self.ep_rank * self.local_experts
         assert intermediate_size % self.moe_tp == 0
         self.inter_local = intermediate_size // self.moe_tp
-        self.w13 = nn.Parameter(torch.zeros(self.local_experts, 2 * self.inter_local, hidden_size, dtype=dtype), requires_grad=False)
+        self.w13 = nn.Parameter(torch.zeros(self.local_experts, (2 if gated else 1) * self.inter_local, hidden_size, dtype=dtype), requires_grad=False)
         self.w2 = nn.Parameter(torch.zeros(self.local_experts, hidden_size, self.inter_local, dtype=dtype), requires_grad=False)
-        self.act = None          # None = silu(gate) * up; ("clamped_glu", limit, alpha) = the clamped GLU (ops/moe_ops.py fused_moe)
+        self.act = None          # None = silu(gate) * up; ("clamped_glu", limit, alpha) = the clamped GLU; ("relu2",) = ungated (ops/moe_ops.py fused_moe)
+        self.gated = gated       # False: one up-projection per expert (``weight_loader`` shard "w3"), needs an ungated ``act``
+        self.weight_input = False      # a routing weight multiplies its expert's input instead of its output
         self.expert_load = None  # EPLB recorder hook
         self.placement = None    # eplb/placement.py ExpertPlacement once experts are replicated / moved; None = contiguous default
         self.rep_table = self.rep_count = None
@@ -93,7 +95,9 @@ class FusedMoE(nn.Module):
         if le < 0 or le >= self.local_experts:
             return
         I, r = self.inter_local, self.moe_tp_rank
-        if shard == "w1":
+        if not self.gated and shard in ("w1", "w3"):
+            param.data[le].copy_(loaded.narrow(0, r * I, I))
+        elif shard == "w1":
             param.data[le, :I].copy_(loaded.narrow(0, r * I, I))
         elif shard == "w3":
             param.data[le, I:].copy_(loaded.narrow(0, r * I, I))
@@ -132,6 +136,7 @@ class FusedMoE(nn.Module):
 
         tp = self.tp
         W = tp.world_size
+        assert not self.weight_input and self.act is None, "all-to-all dispatch: SiLU-GLU experts, weighted outputs"
         assert self.moe_tp == 1 and self.ep_size == W, "all-to-all dispatch needs ep_size == tp_size"
         self._a2a_calls = getattr(self, "_a2a_calls", 0) + 1
         T, H = x.shape
@@ -181,7 +186,7 @@ class FusedMoE(nn.Module):
                 return mgr.forward(self, x, w, ids)
             return self.forward_a2a(x, w, ids)
         tp = self.tp
-        if (tp.world_size > 1 and tp.nvl is not None and x.is_cuda and x.dtype == torch.bfloat16 and x.dim() == 2
+        if (tp.world_size > 1 and self.act is None and tp.nvl is not None and x.is_cuda and x.dtype == torch.bfloat16 and x.dim() == 2
                 and moe_ops._has("moe_grouped_mlp_push") and tp.world_size * x.numel() * 2 <= tp.nvl.slot_bytes):
             from ..environ import envs
             from ..parallel.parallel_state import get_pp_group
@@ -191,7 +196,7 @@ class FusedMoE(nn.Module):
                 # combine kernel pushes the partial sums to every peer; the next RMSNorm reduces them locally
                 off = tp.nvl.moe_push(x, self.w13, self.w2, w, ids.to(torch.int32), self.expert_offset)
                 return PendingAllReduce(tp.nvl, off, x.shape[0], x.shape[1], "push")
-        y = moe_ops.fused_moe(x, self.w13, self.w2, w, ids, self.expert_offset, self.act)
+        y = moe_ops.fused_moe(x, self.w13, self.w2, w, ids, self.expert_offset, self.act, self.weight_input)
         if tp.world_size > 1:
             y = tp.all_reduce(y)
         return y

@@ -154,6 +154,9 @@ def _register_builtins() -> None:
     from . import rumuvik as _rv
 
     register_model("Rumuvik", _rv.RumuvikForCausalLM)
+    from . import mumasun as _mm
+
+    register_model("Mumasun", _mm.MumasunForCausalLM)
     from . import transformers_fallback as _tff
 
     register_model("TransformersForCausalLM", _tff.TransformersForCausalLM)

@@ -125,24 +125,28 @@ def attn_impl() -> int:
 def paged_attention(q, k_cache, v_cache, page_table, req_slots, seq_lens, cu_q, q_lens, max_q_len: int, page_size: int,
                     scale: float, causal: bool = True, window: int = -1, logit_cap: float = 0.0, k_scale: float = 1.0,
                     v_scale: float = 1.0, num_splits: int = 1, workspace=None, tok2req=None, out=None, lse=None,
-                    impl: Optional[int] = None, custom_mask=None, tree_anc=None, slopes=None, log_rates=None, keep_first: int = 0):
+                    impl: Optional[int] = None, custom_mask=None, tree_anc=None, slopes=None, log_rates=None, keep_first: int = 0,
+                    chunk: int = 0, diff=None, diff_dv: int = 0):
     """q [T,Hq,D]; caches [slots,Hkv,D]; cu_q None => decode (q_len 1).  ``slopes`` fp32 [Hq]: a distance bias ``- slopes[h] * (i - j)`` added to
     the (capped) scores, or ``- slopes[h] * ln(1 + log_rates[h] * (i - j))`` when ``log_rates`` fp32 [Hq] is given; ``keep_first``: with a window,
     keys at positions below it stay visible to every later query; all three on the tcgen05 kernels only (``tc_attention_ok`` says whether a call takes them).  ``tree_anc`` int32 [T]: speculative token-tree verification on the
-    tcgen05 kernel (bit k = draft node k is an ancestor-or-self of this query node); ``custom_mask`` = the general (reference-path) form."""
+    tcgen05 kernel (bit k = draft node k is an ancestor-or-self of this query node); ``custom_mask`` = the general (reference-path) form.
+    ``chunk > 0``: a key is visible only in its query's own chunk of that many positions.  ``diff = (lam, post, eps)``: query heads 2h, 2h + 1 are
+    two maps over the same values, combined in the kernel's epilogue (``torch_ref.differential_combine`` over the first ``diff_dv`` columns);
+    the result is [T, Hq / 2, diff_dv].  Both on the tcgen05 kernels only."""
     tree_ok = (tree_anc is not None and _use_native(q) and q.dtype == torch.bfloat16 and attn_impl() == 0 and q.shape[-1] == 128
                and k_cache.dtype == torch.bfloat16 and 128 % (q.shape[1] // k_cache.shape[1]) == 0 and int(max_q_len) <= 32 and window <= 0)
     if _use_native(q) and q.dtype == torch.bfloat16 and (tree_ok or (custom_mask is None and tree_anc is None)):
         if out is None:
-            out = torch.empty(q.shape, dtype=q.dtype, device=q.device)
+            out = torch.empty(q.shape if diff is None else (q.shape[0], q.shape[1] // 2, diff_dv), dtype=q.dtype, device=q.device)
         impl = attn_impl() if impl is None else impl
         D = q.shape[-1]
         Hq, Hkv = q.shape[1], k_cache.shape[1]
         G = Hq // Hkv
         if impl == 0 and (D != 128 or k_cache.dtype != torch.bfloat16 or 128 % G != 0 or page_size < 8 or page_size > 128):
             impl = 1
-        if slopes is not None or keep_first > 0:
-            assert impl == 0 and tree_anc is None, "distance bias / kept first tokens: tcgen05 attention kernels only"
+        if slopes is not None or keep_first > 0 or chunk > 0 or diff is not None:
+            assert impl == 0 and tree_anc is None, "distance bias / kept first tokens / chunks / map pairs: tcgen05 attention kernels only"
         part_o = part_lse = None
         if impl in (0, 2) and num_splits > 1:
             if workspace is None:
@@ -163,9 +167,10 @@ def paged_attention(q, k_cache, v_cache, page_table, req_slots, seq_lens, cu_q, 
         torch.ops.sglb.attn_fwd(q, k_cache, v_cache, out, lse, part_o, part_lse, page_table, req_slots, seq_lens, cu_q, tok2req,
                                 int(max_q_len), int(page_size), int(num_splits), float(scale), bool(causal), int(window),
                                 float(logit_cap), float(k_scale), float(v_scale), int(impl), tree_anc if tree_ok else None, slopes,
-                                log_rates if slopes is not None else None, int(keep_first) if window > 0 else 0)
+                                log_rates if slopes is not None else None, int(keep_first) if window > 0 else 0, int(chunk),
+                                [] if diff is None else [float(diff[0]), float(diff[1]), float(diff[2]), float(diff_dv)])
         return out
-    assert slopes is None and keep_first <= 0, "distance bias / kept first tokens: tcgen05 attention kernels only"
+    assert slopes is None and keep_first <= 0 and chunk <= 0 and diff is None, "distance bias / kept first tokens / chunks / map pairs: tcgen05 kernels only"
     if custom_mask is None and tree_anc is not None:
         custom_mask = torch_ref.tree_anc_to_mask(tree_anc, q_lens, seq_lens)
     r = torch_ref.paged_attention(q, k_cache, v_cache, page_table, req_slots, seq_lens, q_lens, page_size, scale, causal,
@@ -646,31 +651,35 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      seq_lens: torch.Tensor, cu_q: Optional[torch.Tensor], q_lens: Optional[torch.Tensor], max_q_len: int, page_size: int, scale: float,
                      softcap: float = 0.0, window: int = -1, slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
                      dim: int = 0, pad: int = 0, keep_first: int = 0, log_rates: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                     out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, diff=None) -> torch.Tensor:
     """paged grouped-query attention with a tanh score cap, a per-head distance bias, a sliding window and soft-max sinks, for prompt portions
     and decode tokens (csrc/kernels/window_attention.cu; semantics in ``torch_ref.window_attention``).  Returns [T, H, Dv] in q's dtype.
     ``pad > 0``: heads are laid out ``pad`` columns wide in q and in the cache rows; ``dim`` is the key size that counts.
     ``keep_first``: the sequence's first positions stay visible behind the window.  ``log_rates``: the bias is ``slopes_h ln(1 + log_rates_h
     (i - j))``.  ``gate`` [T, H] or [T, H*Dv] (q's dtype, a column view is fine): the output times ``sigmoid(gate)``, per head or per element,
-    then times ``out_scale``, in the kernel's epilogue.  ``out``: a [T, H*Dv] view with unit column stride to write into."""
+    then times ``out_scale``, in the kernel's epilogue.  ``out``: a [T, H*Dv] view with unit column stride to write into.
+    ``chunk``: keys outside the query's own chunk are hidden.  ``diff = (lam, post, eps)``: query heads 2h, 2h + 1 are combined in the epilogue
+    (``torch_ref.differential_combine``); the result is [T, H / 2, Dv]."""
     T, H, D = q.shape
+    Ho = H if diff is None else H // 2
     if pad > 0:
         D = dim
     if (_use_native(q) and q.dtype in (torch.bfloat16, torch.float32) and q.is_contiguous() and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
             and D <= 256 and Dv <= 256 and req_slots.numel() <= 65535 and k_cache.stride(0) == v_cache.stride(0)
             and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape[1] in (H, H * Dv)))):
         if out is None:
-            out = torch.empty(T, H * Dv, dtype=q.dtype, device=q.device)
-        assert out.dtype == q.dtype and out.stride(1) == 1 and out.shape == (T, H * Dv)
+            out = torch.empty(T, Ho * Dv, dtype=q.dtype, device=q.device)
+        assert out.dtype == q.dtype and out.stride(1) == 1 and out.shape == (T, Ho * Dv)
         f = lambda t: None if t is None else t.float().contiguous()
         torch.ops.sglb.window_attention(q, k_cache, v_cache, int(G), int(Dv), page_table, req_slots, seq_lens, cu_q, int(max_q_len), int(page_size),
                                         float(scale), float(softcap), int(window), f(slopes), f(sinks), out, int(D), int(pad), int(keep_first),
-                                        f(log_rates), gate, float(out_scale))
-        return out.view(T, H, Dv) if out.is_contiguous() else out
+                                        f(log_rates), gate, float(out_scale), int(chunk),
+                                        [] if diff is None else [float(diff[0]), float(diff[1]), float(diff[2]), float(Dv)])
+        return out.view(T, Ho, Dv) if out.is_contiguous() else out
     y = torch_ref.window_attention(q, k_cache, v_cache, G, Dv, page_table, req_slots, seq_lens, q_lens, page_size, scale, softcap, window, slopes,
-                                   sinks, dim, pad, keep_first, log_rates, gate, out_scale).to(q.dtype)
+                                   sinks, dim, pad, keep_first, log_rates, gate, out_scale, chunk, diff).to(q.dtype)
     if out is not None:
-        out.copy_(y.view(T, H * Dv))
+        out.copy_(y.view(T, Ho * Dv))
         return out
     return y
 
@@ -847,3 +856,44 @@ def mlstm_readout(y: torch.Tensor, gates: torch.Tensor, H: int, Dv: int, norm_w:
         torch.ops.sglb.mlstm_readout(y, gates, int(H), int(Dv), norm_w, float(eps), gate, out)
         return out
     return torch_ref.mlstm_readout(y, gates, H, Dv, norm_w, eps, gate, out_dtype)
+
+
+# ------------------------------------------------------------------ short-convolution attention preparation / output-normed blocks / fp32 products of model-dtype operands
+def conv_attention_prepare(qkv: torch.Tensor, H: int, G: int, M: int, D: int, Dv: int, conv_w: torch.Tensor, conv_state: torch.Tensor, positions: torch.Tensor,
+                           cu_q: Optional[torch.Tensor], req_slots: torch.Tensor, seq_lens: torch.Tensor, q_norm_w: Optional[torch.Tensor],
+                           k_norm_w: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rot_mult: float, k_cache: torch.Tensor,
+                           v_cache: torch.Tensor, out_cache_loc: torch.Tensor, pad: int = 0) -> torch.Tensor:
+    """short causal convolution over the q / k / v projections, RMS norm and rotation of every (head, map) of q and k, the write of k / v rows into
+    the paged cache and the roll of the convolution state (csrc/kernels/conv_attention.cu; semantics in ``torch_ref.conv_attention_prepare``).
+    Returns q [T, H * M, M * segment] in the cache dtype."""
+    ok = lambda t: t is None or (t.dtype == qkv.dtype and t.is_contiguous())
+    if (_use_native(qkv) and qkv.dtype in (torch.bfloat16, torch.float32) and qkv.stride(1) == 1 and k_cache.dtype == qkv.dtype and v_cache.dtype == qkv.dtype
+            and k_cache.stride(-1) == 1 and v_cache.stride(-1) == 1 and k_cache.stride(0) == v_cache.stride(0) and ok(conv_w) and ok(conv_state)
+            and ok(q_norm_w) and ok(k_norm_w) and D <= 256 and Dv <= 256 and conv_w.shape[1] <= 16 and req_slots.numel() <= 65535):
+        q = torch.empty(qkv.shape[0], H * M, pad if pad > 0 else M * D, dtype=qkv.dtype, device=qkv.device)
+        torch.ops.sglb.conv_attention_prepare(qkv, int(H), int(G), int(M), int(D), int(Dv), conv_w, conv_state, positions, cu_q, req_slots, seq_lens, q_norm_w,
+                                              k_norm_w, float(eps), inv_freq, float(rot_mult), k_cache, v_cache, out_cache_loc, q, int(pad))
+        return q
+    return torch_ref.conv_attention_prepare(qkv, H, G, M, D, Dv, conv_w, conv_state, positions, cu_q, req_slots, seq_lens, q_norm_w, k_norm_w, eps, inv_freq,
+                                            rot_mult, k_cache, v_cache, out_cache_loc, pad)
+
+
+def norm_add_f32(x: Optional[torch.Tensor], src: torch.Tensor, weight: torch.Tensor, eps: float, zero_centred: bool, out_dtype: torch.dtype,
+                 ids: Optional[torch.Tensor] = None):
+    """fp32 stream ``x`` += norm(src) * (1 + w | w); with ``ids`` (int32) a new stream = that of the table rows ``src[ids]`` (csrc/kernels/
+    residual_f32.cu; semantics in ``torch_ref.norm_add_f32``).  Returns (x, x in ``out_dtype``); for fp32 the two are the same tensor."""
+    if x is None:
+        x = torch.empty(ids.shape[0], src.shape[1], dtype=torch.float32, device=src.device)
+    if (_use_native(x) and x.is_contiguous() and src.is_contiguous() and src.dtype in (torch.bfloat16, torch.float32) and weight.dtype == out_dtype
+            and out_dtype in (torch.bfloat16, torch.float32) and (ids is None or ids.dtype == torch.int32)):
+        out = None if out_dtype == torch.float32 else torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        torch.ops.sglb.norm_add_f32(x, src, None if ids is None else ids.contiguous(), weight, out, float(eps), bool(zero_centred))
+        return x, x if out is None else out
+    return x, torch_ref.norm_add_f32(x, src, weight, eps, zero_centred, out_dtype, ids)
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x [T, K] @ w [N, K]^T with an fp32 result: bf16 operands multiply exactly and accumulate in fp32 on the tensor cores (cuBLAS, fp32 output)"""
+    if x.is_cuda and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
+        return torch.mm(x, w.t(), out_dtype=torch.float32)
+    return torch.nn.functional.linear(x.float(), w.float())

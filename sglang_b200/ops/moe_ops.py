@@ -29,9 +29,23 @@ def topk_softmax(router_logits: torch.Tensor, top_k: int, renormalize: bool = Tr
 
 
 def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor,
-              expert_offset: int = 0, act=None) -> torch.Tensor:
-    """``act``: None = silu(gate) * up; ``("clamped_glu", limit, alpha)`` = min(g, limit) * sigmoid(alpha g) * (clamp(u, +-limit) + 1)"""
+              expert_offset: int = 0, act=None, weight_input: bool = False) -> torch.Tensor:
+    """``act``: None = silu(gate) * up; ``("clamped_glu", limit, alpha)`` = min(g, limit) * sigmoid(alpha g) * (clamp(u, +-limit) + 1);
+    ``("relu2",)`` = ungated experts, max(up, 0)^2 with ``w13`` [E, I, H].  ``weight_input``: a routing weight multiplies its expert's input
+    instead of its output (ungated experts)"""
     fn = None
+    assert not weight_input or (act is not None and act[0] == "relu2"), "input weights: ungated experts only"
+    if act is not None and act[0] == "relu2":
+        fn = lambda u: torch.relu(u.float()).square().to(u.dtype)
+        H, I = x.shape[1], w2.shape[2]
+        if (x.is_cuda and x.dtype == torch.bfloat16 and _has("moe_grouped_mlp_relu2") and H % 32 == 0 and I % 32 == 0 and w13.shape[0] <= 512
+                and x.stride(1) == 1 and x.stride(0) % 8 == 0):
+            out = torch.empty_like(x)
+            torch.ops.sglb.moe_grouped_mlp_relu2(x, w13, w2, topk_w, topk_ids, out, expert_offset, weight_input)
+            return out
+        if not x.is_cuda:
+            return torch_ref.fused_moe(x, w13, w2, topk_w, topk_ids, expert_offset, fn, weight_input)
+        return _fused_moe_sorted(x, w13, w2, topk_w, topk_ids, expert_offset, fn, weight_input)
     if act is not None:
         kind, limit, alpha = act
         assert kind == "clamped_glu", kind
@@ -54,7 +68,7 @@ def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torc
     return _fused_moe_sorted(x, w13, w2, topk_w, topk_ids, expert_offset, fn)
 
 
-def _fused_moe_sorted(x, w13, w2, topk_w, topk_ids, expert_offset, act=None):
+def _fused_moe_sorted(x, w13, w2, topk_w, topk_ids, expert_offset, act=None, weight_input=False):
     """sort (token, k) pairs by expert, run one GEMM pair per local expert on its contiguous slice, scatter-add."""
     T, H = x.shape
     E = w13.shape[0]
@@ -67,6 +81,8 @@ def _fused_moe_sorted(x, w13, w2, topk_w, topk_ids, expert_offset, act=None):
     tok = (order // K)
     xs = x.index_select(0, tok[: sum(counts)])
     ws = topk_w.reshape(-1)[order[: sum(counts)]].to(torch.float32)
+    if weight_input:
+        xs = (xs.float() * ws[:, None]).to(x.dtype)
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
     off = 0
     for e, c in enumerate(counts):
@@ -74,7 +90,9 @@ def _fused_moe_sorted(x, w13, w2, topk_w, topk_ids, expert_offset, act=None):
             continue
         h = linear(xs[off:off + c], w13[e])
         h = silu_and_mul(h) if act is None else act(h)
-        y = linear(h, w2[e]).float() * ws[off:off + c, None]
+        y = linear(h, w2[e]).float()
+        if not weight_input:
+            y = y * ws[off:off + c, None]
         out.index_add_(0, tok[off:off + c], y)
         off += c
     return out.to(x.dtype)
@@ -91,6 +109,18 @@ def softmax_bias_route(logits: torch.Tensor, correction, top_k: int, n_real: int
         torch.ops.sglb.moe_softmax_bias_route(logits, None if correction is None else correction.float().contiguous(), int(n_real), w, ids, ident)
         return w, ids, ident
     return torch_ref.softmax_bias_route(logits, correction, top_k, n_real)
+
+
+def sigmoid_route(logits: torch.Tensor, top_k: int, renormalize: bool = False, scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """the ``top_k`` largest logits of every row, weighted ``sigmoid(logit)`` (warp-per-token kernel in csrc/kernels/moe.cu; semantics in
+    ``torch_ref.sigmoid_route``) -> (weights fp32, ids int32)"""
+    T, E = logits.shape
+    if logits.is_cuda and _has("moe_sigmoid_route") and logits.dtype == torch.float32 and logits.stride(1) == 1 and E <= 2048 and top_k <= 32:
+        w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
+        ids = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
+        torch.ops.sglb.moe_sigmoid_route(logits, bool(renormalize), float(scale), w, ids)
+        return w, ids
+    return torch_ref.sigmoid_route(logits, top_k, renormalize, scale)
 
 
 def moe_identity_shared_combine(y: torch.Tensor, h: torch.Tensor, ident_w, shared, shared_logit) -> torch.Tensor:

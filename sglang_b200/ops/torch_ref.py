@@ -258,9 +258,10 @@ def moe_topk_softmax(router_logits: torch.Tensor, top_k: int, renormalize: bool 
 
 
 def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor,
-              expert_offset: int = 0, act=None) -> torch.Tensor:
-    """x [T,H]; w13 [E_local, 2I, H]; w2 [E_local, H, I]; ids are global expert ids; experts outside
-    [expert_offset, expert_offset+E_local) contribute zero (EP)."""
+              expert_offset: int = 0, act=None, weight_input: bool = False) -> torch.Tensor:
+    """x [T,H]; w13 [E_local, 2I, H] ([E_local, I, H] for an ungated ``act``); w2 [E_local, H, I]; ids are global expert ids; experts outside
+    [expert_offset, expert_offset+E_local) contribute zero (EP).  ``weight_input``: a routing weight multiplies its expert's input instead
+    of its output."""
     T, H = x.shape
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
     E = w13.shape[0]
@@ -269,10 +270,11 @@ def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torc
         tok, kk = sel.nonzero(as_tuple=True)
         if tok.numel() == 0:
             continue
-        h = F.linear(x[tok], w13[e])
+        w = topk_w[tok, kk].float()[:, None]
+        h = F.linear((x[tok].float() * w).to(x.dtype) if weight_input else x[tok], w13[e])
         h = silu_and_mul(h) if act is None else act(h)
         y = F.linear(h, w2[e]).float()
-        out.index_add_(0, tok, y * topk_w[tok, kk].float()[:, None])
+        out.index_add_(0, tok, y if weight_input else y * w)
     return out.to(x.dtype)
 
 
@@ -609,12 +611,15 @@ def qk_norm_cache_write(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, posi
 def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, G: int, Dv: int, page_table: torch.Tensor, req_slots: torch.Tensor,
                      seq_lens: torch.Tensor, q_lens: Optional[torch.Tensor], page_size: int, scale: float, softcap: float, window: int,
                      slopes: Optional[torch.Tensor], sinks: Optional[torch.Tensor], dim: int = 0, pad: int = 0, keep_first: int = 0,
-                     log_rates: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
+                     log_rates: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, chunk: int = 0,
+                     diff=None) -> torch.Tensor:
     """grouped-query attention over a paged cache with a tanh score cap, a per-head distance bias, a sliding window and soft-max sinks.
     ``pad > 0``: q is [T, H, pad] and every key / value head occupies ``pad`` cache columns, of which the first ``dim`` / ``Dv`` count.
     ``keep_first``: with a window, the sequence's first ``keep_first`` positions stay visible to every later query.  ``log_rates`` fp32 [H]:
     the distance bias is ``slopes_h * ln(1 + log_rates_h * (i - j))`` instead of linear.  ``gate`` [T, H] or [T, H*Dv]: the output is
-    multiplied by ``sigmoid(gate)`` per head or per element; ``out_scale`` multiplies it once more.
+    multiplied by ``sigmoid(gate)`` per head or per element; ``out_scale`` multiplies it once more.  ``chunk > 0``: key j is visible only when
+    ``i // chunk == j // chunk``.  ``diff = (lam, post, eps)``: query heads 2h, 2h + 1 are combined (``differential_combine``) and the result
+    is [T, H / 2, Dv].
 
     q [T, H, D]; caches [slots, 1, width] with the G key heads in the first ``G*D`` columns (values: ``G*Dv``); query head h reads key head
     ``h // (H // G)``.  score_ij = cap(q_i . k_j * scale) - slopes_h * (i - j) with cap(s) = softcap * tanh(s / softcap) (``softcap <= 0``:
@@ -634,6 +639,8 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         if ql <= 0:
             continue
         lo = 0 if window <= 0 else max(0, L - ql - window + 1)
+        if chunk > 0:
+            lo = (L - ql) // chunk * chunk
         pos = torch.arange(lo, L, device=q.device)
         if keep_first > 0 and lo > 0:
             pos = torch.cat([torch.arange(0, min(keep_first, lo), device=q.device), pos])
@@ -653,6 +660,8 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         if window > 0:
             far = dist >= window
             hide = hide | (far & (pos[None, :] >= keep_first) if keep_first > 0 else far)
+        if chunk > 0:
+            hide = hide | (qpos // chunk != pos[None, :] // chunk)
         s = s.masked_fill(hide[None], float("-inf"))
         if sinks is not None:
             s = torch.cat([s, sinks.float()[:, None, None].expand(H, ql, 1)], -1)
@@ -662,6 +671,8 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     if gate is not None:
         g = torch.sigmoid(gate.float())
         out = out * (g[:, :, None] if g.shape[1] == H else g.view(T, H, Dv))
+    if diff is not None:
+        out = differential_combine(out, *diff)
     return out * out_scale if out_scale != 1.0 else out
 
 
@@ -678,6 +689,71 @@ def softmax_bias_route(logits: torch.Tensor, correction: Optional[torch.Tensor],
 
 
 # ------------------------------------------------------------------ Resatar mechanisms: attention preparation (projection-wide norm, partial rotation, value mixing), selective scan
+def sigmoid_route(logits: torch.Tensor, top_k: int, renormalize: bool = False, scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """the ``top_k`` largest logits of every row, weighted ``sigmoid(logit)`` (divided by their sum with ``renormalize``) times ``scale``"""
+    z, ids = logits.float().topk(top_k, dim=-1)
+    w = torch.sigmoid(z)
+    if renormalize:
+        w = w / w.sum(-1, keepdim=True)
+    return (w * scale).contiguous(), ids.to(torch.int32).contiguous()
+
+
+def norm_add_f32(x: torch.Tensor, src: torch.Tensor, weight: torch.Tensor, eps: float, zero_centred: bool, out_dtype: torch.dtype,
+                 ids: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x (fp32, in place) += norm(src) * (1 + w | w), or x = that of the table rows ``src[ids]``; returns x in ``out_dtype``"""
+    s = (src if ids is None else src[ids.long()]).float()
+    y = s * torch.rsqrt(s.pow(2).mean(-1, keepdim=True) + eps) * (1.0 + weight.float() if zero_centred else weight.float())
+    if ids is None:
+        x.add_(y)
+    else:
+        x.copy_(y)
+    return x.to(out_dtype)
+
+
+def differential_combine(o: torch.Tensor, lam: float, post: float, eps: float) -> torch.Tensor:
+    """o [T, 2H, Dv], rows 2h and 2h + 1 the two maps of head h -> unit_rms(o_2h - lam o_2h+1) * post, fp32 [T, H, Dv]"""
+    a = o.float().unflatten(1, (-1, 2))
+    d = a[:, :, 0] - lam * a[:, :, 1]
+    return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * post
+
+
+def conv_attention_prepare(qkv: torch.Tensor, H: int, G: int, M: int, D: int, Dv: int, conv_w: torch.Tensor, conv_state: torch.Tensor,
+                           positions: torch.Tensor, cu_q, req_slots: torch.Tensor, seq_lens: torch.Tensor, q_norm_w, k_norm_w, eps: float,
+                           inv_freq, rot_mult: float, k_cache: torch.Tensor, v_cache: torch.Tensor, out_cache_loc: torch.Tensor,
+                           pad: int = 0) -> torch.Tensor:
+    """projection rows ``qkv`` [T, >= C] = [q (H*M*D) | k (G*M*D) | v (G*Dv)] -> q rows for the attention kernel, k and v rows in the cache:
+
+    * a causal convolution over time per channel (``conv_w`` [C, taps], tap ``taps - 1`` = the current token; ``conv_state`` [slots, C, taps - 1]
+      is each request's last inputs, rolled forward in place);
+    * ``q_norm_w`` / ``k_norm_w`` [D]: RMS norm of every (head, map), times the weight;
+    * ``inv_freq`` fp32 [R/2]: the first R coordinates turned by ``position * inv_freq[i]``, i paired with i + R/2, sine and cosine times
+      ``rot_mult``;
+    * k head g takes M segments side by side; q is [T, H * M, M * segment] whose row ``h * M + m`` holds map m of head h in segment m and
+      zeros elsewhere.  A segment is D columns, or ``pad / M`` with ``pad`` (values then occupy ``pad`` columns, zeros behind them)."""
+    T, C = qkv.shape[0], (H + G) * M * D + G * Dv
+    x, taps = qkv[:, :C], conv_w.shape[1]
+    u = causal_conv1d(x, conv_w, None, conv_state, cu_q, req_slots, seq_lens, silu=False) if taps > 1 else x.float() * conv_w[:, 0].float()
+    q, k, v = u[:, :H * M * D].reshape(T, H, M, D), u[:, H * M * D:(H + G) * M * D].reshape(T, G, M, D), u[:, (H + G) * M * D:].reshape(T, G, Dv)
+    if q_norm_w is not None:
+        nrm = lambda t, w: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        q, k = nrm(q, q_norm_w), nrm(k, k_norm_w)
+    if inv_freq is not None:
+        half = inv_freq.numel()
+        ang = (positions.float()[:, None] * inv_freq.float()[None, :])[:, None, None, :]
+        c, s = torch.cos(ang) * rot_mult, torch.sin(ang) * rot_mult
+        turn = lambda t: torch.cat([t[..., :half] * c - t[..., half:2 * half] * s, t[..., half:2 * half] * c + t[..., :half] * s, t[..., 2 * half:]], -1)
+        q, k = turn(q), turn(k)
+    seg, wv = (pad // M, pad) if pad > 0 else (D, Dv)
+    zp = lambda t, n: torch.nn.functional.pad(t, (0, n - t.shape[-1]))
+    loc = out_cache_loc.long()
+    k_cache[loc, 0, :G * M * seg] = zp(k, seg).reshape(T, G * M * seg).to(k_cache.dtype)
+    v_cache[loc, 0, :G * wv] = zp(v, wv).reshape(T, G * wv).to(v_cache.dtype)
+    qo = torch.zeros(T, H, M, M, seg, dtype=k_cache.dtype, device=qkv.device)
+    for m in range(M):
+        qo[:, :, m, m] = zp(q[:, :, m], seg).to(k_cache.dtype)
+    return qo.view(T, H * M, M * seg)
+
+
 def attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, positions: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       out_cache_loc: torch.Tensor, q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
                       inv_freq: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0, pad: int = 0,
