@@ -1,0 +1,212 @@
+"""Mumasun CUDA kernels against their fp32 PyTorch references (``ops/torch_ref.py``) and the engine on CUDA against the plain oracle."""
+import numpy as np
+import pytest
+import torch
+
+from sglang_b200 import ops
+from sglang_b200.layers.latent_attention import yarn_inv_freq
+from sglang_b200.ops import moe_ops, torch_ref
+
+pytestmark = pytest.mark.gpu
+
+DEV = "cuda"
+
+
+def _need():
+    if not torch.cuda.is_available():
+        pytest.skip("needs a GPU")
+    assert ops.load_native(), "the CUDA extension must be built on a GPU box"
+
+
+def _i32(x, dev=DEV):
+    return torch.tensor(x, dtype=torch.int32, device=dev)
+
+
+def _tol(dtype, f32=(1e-5, 1e-5), bf=(2e-2, 2e-2)):
+    r, a = bf if dtype == torch.bfloat16 else f32
+    return dict(rtol=r, atol=a)
+
+
+def _pages(n_req, max_len, ps, g):
+    """page table whose pages lie scattered over the pool; rows 1 .. n_req"""
+    per = (max_len + ps - 1) // ps
+    n_pages = n_req * per + 3
+    pt = torch.zeros(n_req + 1, per + 1, dtype=torch.int32)
+    perm = torch.randperm(n_pages - 1, generator=g) + 1
+    for r in range(n_req):
+        pt[r + 1, :per] = perm[r * per:(r + 1) * per].int()
+    return pt, n_pages
+
+
+def _slots(pt, row, positions, ps):
+    return [int(pt[row, p // ps]) * ps + p % ps for p in positions]
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("W", [24, 250, 1024, 5000])
+def test_norm_add(dtype, W):
+    _need()
+    g = torch.Generator().manual_seed(W)
+    x, y = torch.randn(7, W, generator=g), torch.randn(7, W, generator=g).to(dtype)
+    w = (torch.randn(W, generator=g) * 0.2).to(dtype)
+    for zc in (True, False):
+        r = x.clone()
+        ref = torch_ref.norm_add_f32(r, y, w, 1e-5, zc, dtype)
+        gx, gh = ops.norm_add_f32(x.clone().to(DEV), y.to(DEV), w.to(DEV), 1e-5, zc, dtype)
+        torch.testing.assert_close(gx.cpu(), r, rtol=1e-5, atol=1e-5)
+        torch.testing.assert_close(gh.cpu().float(), ref.float(), **_tol(dtype, bf=(8e-3, 1e-3)))
+        assert gh.dtype == dtype and (dtype != torch.float32 or gh is gx)
+    table, ids = torch.randn(11, W, generator=g).to(dtype), _i32([3, 10, 0, 3])
+    r = torch.empty(4, W)
+    torch_ref.norm_add_f32(r, table, w, 1e-5, True, dtype, ids.cpu())
+    gx, gh = ops.norm_add_f32(None, table.to(DEV), w.to(DEV), 1e-5, True, dtype, ids)
+    torch.testing.assert_close(gx.cpu(), r, rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(gh.cpu().float(), r, **_tol(dtype, bf=(8e-3, 1e-3)))
+
+
+@pytest.mark.parametrize("E,K", [(1, 1), (8, 1), (8, 8), (40, 3), (300, 32), (2048, 2)])
+def test_sigmoid_route(E, K):
+    _need()
+    g = torch.Generator().manual_seed(E + K)
+    z = torch.randn(33, E, generator=g) * 3
+    z[5] += 60.0                                                       # saturated scores: the choice still follows the logits
+    for renorm, scale in ((False, 1.0), (True, 2.5)):
+        w0, i0 = torch_ref.sigmoid_route(z, K, renorm, scale)
+        w1, i1 = moe_ops.sigmoid_route(z.to(DEV), K, renorm, scale)
+        assert torch.equal(i1.cpu(), i0)
+        torch.testing.assert_close(w1.cpu(), w0, rtol=1e-5, atol=1e-7)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("T,W,I,E,K", [(1, 64, 32, 4, 1), (5, 96, 64, 6, 2), (300, 256, 96, 8, 1), (700, 128, 160, 5, 5), (40, 72, 40, 3, 2)])
+def test_experts_with_weighted_inputs(T, W, I, E, K, dtype):
+    _need()
+    g = torch.Generator().manual_seed(T)
+    x = torch.randn(T, W, generator=g).to(dtype)
+    w1, w2 = (torch.randn(E, I, W, generator=g) * W ** -0.5).to(dtype), (torch.randn(E, W, I, generator=g) * I ** -0.5).to(dtype)
+    rw, ids = torch_ref.sigmoid_route(torch.randn(T, E, generator=g) * 2, K)
+    for win in (True, False):
+        act = lambda u: torch.relu(u.float()).square()
+        ref = torch_ref.fused_moe(x.float(), w1.float(), w2.float(), rw, ids, 0, act, win)
+        got = moe_ops.fused_moe(x.to(DEV), w1.to(DEV), w2.to(DEV), rw.to(DEV), ids.to(DEV), 0, ("relu2",), win)
+        assert got.dtype == dtype
+        torch.testing.assert_close(got.cpu().float(), ref, **_tol(dtype, f32=(1e-4, 1e-4), bf=(3e-2, 5e-2)))
+    a = moe_ops.fused_moe(x.to(DEV), w1.to(DEV), w2.to(DEV), rw.to(DEV), ids.to(DEV), 0, ("relu2",), True)
+    b = moe_ops.fused_moe(x[:1].to(DEV), w1.to(DEV), w2.to(DEV), rw[:1].to(DEV), ids[:1].to(DEV), 0, ("relu2",), True)
+    torch.testing.assert_close(a[:1].float(), b.float(), **_tol(dtype, f32=(1e-5, 1e-5), bf=(2e-2, 2e-2)))          # what else is in the batch does not matter
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,M,D,Dv,rot,taps,pad", [(4, 2, 2, 64, 128, 64, 3, 0), (4, 2, 2, 64, 128, 64, 3, 128), (6, 3, 2, 24, 40, 16, 2, 128), (3, 1, 2, 7, 9, 6, 5, 0),
+                                                     (2, 2, 2, 130, 200, 20, 4, 0), (2, 1, 1, 16, 16, 0, 1, 0), (4, 4, 2, 33, 65, 0, 16, 0), (2, 1, 1, 100, 96, 100, 4, 128)])
+def test_conv_attention_prepare(H, G, M, D, Dv, rot, taps, pad, dtype):
+    """ragged portions (single tokens among them, cached history, empty requests), then decode steps of all requests: q rows, cache rows and state"""
+    _need()
+    if pad and D > pad // M:
+        pytest.skip("does not fit the padded layout")
+    g = torch.Generator().manual_seed(H * 100 + D)
+    C, ps = (H + G) * M * D + G * Dv, 8
+    seg, wv = (pad // M, pad) if pad else (D, Dv)
+    width = max(G * M * seg, G * wv) + 3
+    width += -width % 8
+    f, mult = yarn_inv_freq(rot, 500.0, {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}) if rot else (None, 1.0)
+    w = (torch.randn(C, taps, generator=g) * 0.5).to(dtype)
+    nq, nk = (torch.rand(D, generator=g) + 0.5).to(dtype), (torch.rand(D, generator=g) + 0.5).to(dtype)
+    pt, n_pages = _pages(5, 400, ps, g)
+    mk = lambda: (torch.full((n_pages * ps, 1, width), 0.25, dtype=dtype), torch.full((n_pages * ps, 1, width), 0.25, dtype=dtype))
+    (k0, v0), st0 = mk(), torch.randn(7, C, max(1, taps - 1), generator=g).to(dtype)          # a used pool and state: fresh requests must not see it
+    k1, v1, st1 = k0.to(DEV), v0.to(DEV), st0.to(DEV)
+    done = [0, 0, 0, 0, 0]
+    steps = [[40, 1, 0, 3, 2], [1, 17, 2, 0, 300], [5, 2, 1, 1, 3]] + [None] * 3                # None: one token of every request (decode layout)
+    if dtype == torch.float32:
+        steps += [[2, 90, 1, 1, 1]]
+    for n_step, lens in enumerate(steps):
+        ql = lens or [1] * 5
+        T = sum(ql)
+        x = torch.randn(T, C + 5, generator=g).to(dtype)[:, :C] if n_step % 2 else torch.randn(T, C, generator=g).to(dtype)
+        pos = [p for b in range(5) for p in range(done[b], done[b] + ql[b])]
+        loc = [s for b in range(5) for s in _slots(pt, b + 1, range(done[b], done[b] + ql[b]), ps)]
+        done = [a + b for a, b in zip(done, ql)]
+        cu = _i32(np.concatenate([[0], np.cumsum(ql)]).tolist()) if lens else None
+        slots, sl = _i32([1, 4, 2, 6, 3]), _i32(done)
+        c = lambda t: None if t is None else t.cpu()
+        args = lambda dev: (f if dev == "cpu" or f is None else f.to(DEV), mult)
+        q0 = torch_ref.conv_attention_prepare(x, H, G, M, D, Dv, w, st0, _i32(pos, "cpu"), c(cu), c(slots), c(sl), nq, nk, 1e-5, *args("cpu"), k0, v0, _i32(loc, "cpu"), pad)
+        q1 = ops.conv_attention_prepare(x.to(DEV) if x.is_contiguous() else torch.nn.functional.pad(x, (0, 5)).to(DEV)[:, :C], H, G, M, D, Dv, w.to(DEV), st1, _i32(pos), cu,
+                                        slots, sl, nq.to(DEV), nk.to(DEV), 1e-5, *args("cuda"), k1, v1, _i32(loc), pad)
+        t = _tol(dtype, f32=(2e-4, 2e-4), bf=(1e-2, 1e-2))
+        torch.testing.assert_close(q1.cpu().float(), q0.float(), **t)
+        torch.testing.assert_close(k1.cpu().float(), k0.float(), **t)
+        torch.testing.assert_close(v1.cpu().float(), v0.float(), **t)
+        if taps > 1:
+            assert torch.equal(st1.cpu(), st0), n_step                        # the state holds projections: moved, never computed
+
+
+def _attention_case(H, G, D, Dv, lens, cached, ps, chunk, dtype, tc, seed=0, decode=False, splits=1):
+    """differential attention over a paged cache of random rows: (kernel result, fp32 reference), both [T, H, Dv]"""
+    g = torch.Generator().manual_seed(seed)
+    M, pad = 2, 128 if tc else 0
+    seg, wv = (64, 128) if tc else (D, Dv)
+    B, T = len(lens), sum(lens)
+    tot = [a + b for a, b in zip(lens, cached)]
+    pt, n_pages = _pages(B, max(tot), ps, g)
+    width = G * 128 + 16 if tc else max(G * M * D, G * Dv)
+    kc, vc = torch.zeros(n_pages * ps, 1, width), torch.zeros(n_pages * ps, 1, width)
+    for m in range(G * M):
+        kc[:, 0, m * seg:m * seg + D] = torch.randn(n_pages * ps, D, generator=g)
+    for m in range(G):
+        vc[:, 0, m * wv:m * wv + Dv] = torch.randn(n_pages * ps, Dv, generator=g)
+    q = torch.zeros(T, H, M, M, seg)
+    for m in range(M):
+        q[:, :, m, m, :D] = torch.randn(T, H, D, generator=g)
+    q = q.view(T, H * M, M * seg).to(dtype)
+    kc, vc = kc.to(dtype), vc.to(dtype)
+    rows, sl, ql = _i32(list(range(1, B + 1)), "cpu"), _i32(tot, "cpu"), _i32(lens, "cpu")
+    diff, scale = (0.7, 0.6, 1e-5), D ** -0.5
+    ref = torch_ref.window_attention(q.float(), kc.float(), vc.float(), G, Dv, pt, rows, sl, ql, ps, scale, 0.0, -1, None, None, 2 * seg, pad, chunk=chunk, diff=diff)
+    cu = None if decode else _i32(np.concatenate([[0], np.cumsum(lens)]).tolist())
+    a = [t.to(DEV) for t in (q, kc, vc, pt, rows, sl, ql)]
+    if tc:
+        k4, v4 = (t[:, 0, :G * 128].unflatten(-1, (G, 128)) for t in a[1:3])
+        assert ops.tc_attention_ok(a[0], k4, v4, ps)
+        got = ops.paged_attention(a[0], k4, v4, a[3], a[4], a[5], cu, a[6], max(lens), ps, scale, num_splits=splits, chunk=chunk, diff=diff, diff_dv=Dv)
+    else:
+        got = ops.window_attention(a[0], a[1], a[2], G, Dv, a[3], a[4], a[5], cu, a[6], max(lens), ps, scale, dim=2 * D, chunk=chunk, diff=diff)
+    return got.cpu().float(), ref
+
+
+CHUNKS = (0, 48, 64, 100, 1000)
+
+
+@pytest.mark.parametrize("chunk", CHUNKS)
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 32, 48), (6, 1, 9, 7), (3, 3, 100, 130), (40, 2, 16, 16)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_general_attention_kernel(H, G, D, Dv, dtype, chunk):
+    _need()
+    for lens, cached, dec in (([70, 1, 130, 5], [0, 99, 30, 62], False), ([1] * 5, [0, 47, 48, 199, 63], True)):
+        got, ref = _attention_case(H, G, D, Dv, lens, cached, 16, chunk, dtype, False, seed=H, decode=dec)
+        torch.testing.assert_close(got, ref, **_tol(dtype, f32=(2e-4, 2e-5), bf=(3e-2, 1.5e-2)))
+
+
+@pytest.mark.parametrize("chunk", CHUNKS)
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 64, 128), (16, 4, 64, 128), (2, 2, 32, 40), (8, 1, 48, 33), (32, 1, 64, 64)])
+def test_tensor_core_kernels(H, G, D, Dv, chunk):
+    """the tcgen05 kernels (prompt tiles, decode with and without split keys; group sizes that take the query-major kernel in decode) against the
+    reference"""
+    _need()
+    tol = dict(rtol=4e-2, atol=4e-2)
+    for ps in (16, 64):
+        got, ref = _attention_case(H, G, D, Dv, [150, 1, 333, 5], [0, 99, 130, 62], ps, chunk, torch.bfloat16, True, seed=H)
+        torch.testing.assert_close(got, ref, **tol)
+    for splits in (1, 4):
+        got, ref = _attention_case(H, G, D, Dv, [1] * 6, [0, 47, 48, 799, 63, 300], 64, chunk, torch.bfloat16, True, seed=H, decode=True, splits=splits)
+        torch.testing.assert_close(got, ref, **tol)
+
+
+def test_tensor_core_kernels_many_items():
+    """more work items than resident CTAs: the persistent launches, with pairs of maps and chunk edges inside tiles"""
+    _need()
+    got, ref = _attention_case(16, 4, 64, 128, [400, 300, 513, 2, 250], [0, 100, 31, 700, 5], 64, 96, torch.bfloat16, True, seed=1)
+    torch.testing.assert_close(got, ref, rtol=4e-2, atol=4e-2)
+    got, ref = _attention_case(8, 8, 64, 96, [1] * 60, [(37 * i) % 500 for i in range(60)], 64, 200, torch.bfloat16, True, seed=2, decode=True)
+    torch.testing.assert_close(got, ref, rtol=4e-2, atol=4e-2)
