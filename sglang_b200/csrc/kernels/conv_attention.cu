@@ -128,7 +128,7 @@ __global__ void __launch_bounds__(CA_NT) conv_attention_prepare_kernel(const Con
     bool enter = true;
     for (int t = t0; t < t1; ++t) {
       if (p.cu_q) {
-        while (t >= p.cu_q[b + 1]) { ++b; enter = true; }
+        while (b + 1 < p.B && t >= p.cu_q[b + 1]) { ++b; enter = true; }      // tokens behind the last request (padded batches) count to it
       } else if (t > t0) {
         b = t;
         enter = true;

@@ -526,11 +526,12 @@ class ModelRunner:
         self.step_counter += 1
         # the captured sampler sees only the static tensors: anything that needs per-request host state (penalties, logit bias, active
         # min_new_tokens -> EOS mask, per-request seeds, hidden-state return) takes the eager path (ScheduleBatch.needs_host_state)
-        use_graph = decode and self.graphs and not sb.return_logprob and not sb.has_grammar and sb.spec_info is None and \
+        wants_rows = sb.logit_rows is not None and len(sb.logit_rows) > 0          # a replayed step that hands logits back: the graphs keep none
+        use_graph = decode and self.graphs and not wants_rows and not sb.return_logprob and not sb.has_grammar and sb.spec_info is None and \
             B <= self.graph_bs[-1] and not sb.needs_host_state() and (sb.out_cache_loc_swa is None or self.graphs[self.graph_bs[-1]].has_swa)
         if use_graph:
             return self._forward_graph(sb)
-        if self.prefill_graphs and not decode and self._prefill_graph_eligible(sb):
+        if self.prefill_graphs and not decode and not wants_rows and self._prefill_graph_eligible(sb):
             return self._forward_prefill_graph(sb)
         fb = self.packer.build(sb, self.page_table, self.page_size, self.kv_pool, self.next_token_buf, ops.apply_pt_delta)
         fb.swa_pt_offset = getattr(self, "swa_pt_offset", 0)

@@ -210,3 +210,141 @@ def test_tensor_core_kernels_many_items():
     torch.testing.assert_close(got, ref, rtol=4e-2, atol=4e-2)
     got, ref = _attention_case(8, 8, 64, 96, [1] * 60, [(37 * i) % 500 for i in range(60)], 64, 200, torch.bfloat16, True, seed=2, decode=True)
     torch.testing.assert_close(got, ref, rtol=4e-2, atol=4e-2)
+
+
+@pytest.mark.parametrize("dtype,D,Dv,tc", [(torch.float32, 4, 6, False), (torch.bfloat16, 48, 72, True), (torch.bfloat16, 64, 128, True), (torch.bfloat16, 72, 40, False)])
+def test_chunk_edges_and_far_keys_on_the_kernels(dtype, D, Dv, tc):
+    from test_mumasun import LayerBench, check_chunk_edges
+
+    _need()
+    assert (LayerBench(2, 1, D, Dv, 1.0, 0.3, dtype=dtype).m.pad == 128) == tc
+    check_chunk_edges(DEV, dtype, 16, D, Dv, 2e-3 if dtype == torch.float32 else 4e-2)
+
+
+def _engine_case(tmp_path, dtype, cfg, seed, tol, gen=True, quantile=1.0, **kw):
+    """whole prompts, portions, decoding, unequal batches and reuse on CUDA against the oracle.  fp32 bounds every logit; bf16 bounds, per position, the
+    root mean square of the difference over the vocabulary against that of the logits.  ``quantile`` < 1: stacks of tiny or drawn sizes, where in
+    bf16 a router's close call may fall the other way or a norm over a handful of numbers is badly conditioned: that quantile is bounded, and
+    the mean"""
+    from test_mumasun import Harness, _tokens
+
+    h = Harness(tmp_path, cfg, seed=seed, slots=4, max_tokens=1024, device="cuda", dtype=dtype, page=16, **kw)
+    V = cfg["vocab"]
+    a, b, c = _tokens(150, V, 1), _tokens(41, V, 2), _tokens(3, V, 3)
+    ra, rb, rc = h.oracle(a), h.oracle(b), h.oracle(c)
+    errs = []
+
+    def close(x, y):
+        if dtype == "float32":
+            err = np.abs(x - y).max() / max(1.0, float(np.sqrt((y ** 2).mean())))
+            assert float(err) < tol, float(err)
+            return
+        d, r = x - y, y - y.mean(-1, keepdims=True)
+        d = d - d.mean(-1, keepdims=True)
+        errs.append(np.sqrt((d ** 2).mean(-1)) / np.sqrt((r ** 2).mean(-1) + 1e-12))
+
+    close(h.step([("a", a, range(len(a)))], ["a"]), ra)                                            # whole
+    close(h.run_cut("a2", a, [100, 2, 17]), ra)                                                    # portions, then token by token
+    out = h.step([("a", a[:90], range(90)), ("b", b[:7], range(7)), ("c", c, range(3))], ["c"])    # unequal batch
+    close(out[:90], ra[:90]); close(out[90:97], rb[:7]); close(out[97:], rc)
+    out = h.step([("a", a[90:], range(60)), ("b", b[7:8], range(1))], ["a"])
+    close(out[:60], ra[90:]); close(out[60:], rb[7:8])
+    out = h.step([("b", b[8:], range(len(b) - 8)), ("d", c, range(3))], ["b", "d"])                # "d" reuses a freed slot and pages
+    close(out[:len(b) - 8], rb[8:]); close(out[len(b) - 8:], rc)
+    if errs:
+        err = np.concatenate(errs)
+        assert float(np.quantile(err, quantile)) < tol and float(err.mean()) < 0.5 * tol, (float(np.quantile(err, quantile)), float(err.mean()), float(err.max()))
+    if dtype == "float32" and gen:  # greedy generation through the engine's own entry point, scheduler and sampler
+        prompts = [b[:9], c]
+        outs = h.eng.generate(input_ids=prompts, sampling_params={"max_new_tokens": 6, "temperature": 0, "ignore_eos": True})
+        for pr, o in zip(prompts, outs):
+            seq = list(pr)
+            for _ in range(6):
+                seq.append(int(h.oracle(seq)[-1].argmax()))
+            assert o["output_ids"] == seq[len(pr):]
+    h.close()
+
+
+def _wide():
+    """lane-friendly sizes: bf16 layers with map pairs in groups of 8, 2 and 4 take the tcgen05 kernels, the ones with three query heads per key head or
+    wide maps the general kernel"""
+    from test_mumasun import L, _cfg, _mix, _moe
+
+    return _cfg([L(_mix(heads=8, kv_heads=2, dim=64, vdim=128, rot_dims=64, base=1e4, scale=0.2, chunk=48), _moe(64, 8, 1)),
+                 L(_mix(heads=2, kv_heads=2, dim=48, vdim=64, rot_dims=32, base=1e4, scale=0.2, chunk=100, conv=2), _moe(96, 4, 2)),
+                 L(_mix(heads=6, kv_heads=2, dim=32, vdim=48, rot_dims=8, scale=0.25, chunk=30), None),
+                 L(_mix(heads=4, kv_heads=2, dim=96, vdim=64, rot_dims=96, scale=0.1, chunk=0, conv=4), _moe(40, 3, 3))], width=128, vocab=256)
+
+
+def test_engine_on_cuda_fp32(tmp_path):
+    from test_mumasun import MIXED
+
+    _need()
+    _engine_case(tmp_path, "float32", MIXED, 1, 3e-4)
+
+
+def test_engine_on_cuda_bf16(tmp_path):
+    from test_mumasun import MIXED
+
+    _need()
+    _engine_case(tmp_path, "bfloat16", MIXED, 2, 0.2, quantile=0.9)
+
+
+def test_engine_on_cuda_lane_friendly_sizes_fp32(tmp_path):
+    _need()
+    _engine_case(tmp_path, "float32", _wide(), 3, 3e-4)
+
+
+def test_engine_on_cuda_lane_friendly_sizes_bf16(tmp_path):
+    _need()
+    _engine_case(tmp_path, "bfloat16", _wide(), 4, 0.1, quantile=0.95)
+
+
+def test_tensor_core_route_agrees_with_the_general_kernel(tmp_path, monkeypatch):
+    from sglang_b200.layers.differential_attention import DifferentialAttention
+    from test_mumasun import Harness
+
+    _need()
+    h = Harness(tmp_path, _wide(), seed=5, slots=2, max_tokens=512, device="cuda", dtype="bfloat16", page=16)
+    pads = [b.mix.pad for b in h.model.model.all_layers]
+    h.close()
+    assert pads == [128, 128, 0, 0]
+    monkeypatch.setattr(DifferentialAttention, "tc_route", False)
+    _engine_case(tmp_path / "general", "bfloat16", _wide(), 5, 0.1, quantile=0.95)
+
+
+@pytest.mark.parametrize("seed", [11, 12, 13, 14])
+def test_engine_on_cuda_randomly_drawn_stacks_fp32(tmp_path, seed):
+    from test_mumasun import drawn_config
+
+    _need()
+    _engine_case(tmp_path, "float32", drawn_config(seed, friendly=seed % 2 == 0), seed, 2e-3, gen=False)
+
+
+@pytest.mark.parametrize("seed", [21, 22, 31, 32])
+def test_engine_on_cuda_randomly_drawn_stacks_bf16(tmp_path, seed):
+    """friendly sizes, and sizes that are no multiples of the vector widths: every kernel takes its scalar path, the GEMMs their general one"""
+    from test_mumasun import drawn_config
+
+    _need()
+    _engine_case(tmp_path, "bfloat16", drawn_config(seed, friendly=seed < 30), seed, 0.25, quantile=0.9)
+
+
+def test_captured_decode_steps_agree_with_eager_ones(tmp_path):
+    """greedy bf16 generation with CUDA graphs (padded batch sizes, slots that are used again) against the same engine without them"""
+    from test_mumasun import Harness, _tokens
+
+    _need()
+    cfg = _wide()
+    prompts = [_tokens(n, 256, 300 + n) for n in (70, 3, 25, 44, 1, 60, 47)]
+    sp = {"max_new_tokens": 40, "temperature": 0, "ignore_eos": True}
+    outs = []
+    for graphs in (True, False):
+        h = Harness(tmp_path / str(graphs), cfg, seed=6, slots=3, max_tokens=1024, device="cuda", dtype="bfloat16", page=16, disable_cuda_graph=not graphs)
+        r = h.sched.worker.runner if hasattr(h.sched.worker, "runner") else h.sched.worker
+        assert bool(r.graphs) == graphs
+        outs.append([o["output_ids"] for o in h.eng.generate(input_ids=prompts, sampling_params=sp)])
+        assert (r.graph_launches > 0) == graphs
+        h.sched.check_invariants()
+        h.close()
+    assert outs[0] == outs[1]
