@@ -27,6 +27,7 @@ namespace {
 
 constexpr int CA_NT = 256;            // 8 warps
 constexpr int CA_MAX_N = 256;         // widest head
+constexpr int CA_VW = 64;             // columns of a value unit in the four-column kernel
 
 struct ConvPrepParams {
   const void* qkv; int ld;
@@ -38,7 +39,7 @@ struct ConvPrepParams {
   const float* inv_freq; int half; float rot_mult;
   void* kc; void* vc; size_t ldc; const int* loc;
   void* q_out; int seg, wv;           // segment of a map, width of a value head
-  int run, units, units_per_cta;
+  int run, units, units_per_cta, vpieces;         // vpieces: value units per head (four-column kernel)
 };
 
 template <typename T> __device__ __forceinline__ float ca_ld(const T* p);
@@ -251,6 +252,210 @@ __global__ void __launch_bounds__(CA_NT) conv_attention_prepare_kernel(const Con
   }
 }
 
+// four columns of a row
+__device__ __forceinline__ void ca_ld4(const float* p, float (&v)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void ca_ld4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 a = *reinterpret_cast<const uint2*>(p);
+  v[0] = bf16_lo(a.x); v[1] = bf16_hi(a.x); v[2] = bf16_lo(a.y); v[3] = bf16_hi(a.y);
+}
+__device__ __forceinline__ void ca_st4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void ca_st4(__nv_bfloat16* p, const float (&v)[4]) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3])); }
+
+// The same work for maps at most 64 wide, at most four taps and sizes in multiples of four: a half-warp owns a unit (a (head, map) of q or k, or a
+// 64-column piece of a value head), a lane four neighbouring columns; a group of AHEAD tokens that lies in one request convolves straight from
+// the loaded rows, with no moves between them, and its norms and rotations run side by side.
+template <typename T, int AHEAD>
+__global__ void __launch_bounds__(CA_NT) conv_attention_prepare_x4_kernel(const ConvPrepParams p) {
+  constexpr int KM = 4;
+  extern __shared__ float sm[];
+  float* s_cs = sm;                                         // [run][half][cos, sin]
+  int* s_loc = reinterpret_cast<int*>(s_cs + (size_t)p.run * p.half * 2);      // [run] cache slots
+  int* s_b = s_loc + p.run;                                 // request of the run's first token
+  const int t0 = blockIdx.x * p.run, t1 = min(p.T, t0 + p.run);
+  const int lane = threadIdx.x & 31, hl = lane & 15, col = 4 * hl;
+  if (threadIdx.x == 0) {
+    int b = t0;
+    if (p.cu_q) {                                           // last request that starts at or before t0
+      int lo = 0, hi = p.B - 1;
+      while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (p.cu_q[mid] <= t0) lo = mid; else hi = mid - 1;
+      }
+      b = lo;
+    }
+    *s_b = b;
+  }
+  for (int i = threadIdx.x; i < t1 - t0; i += CA_NT) s_loc[i] = p.loc[t0 + i];
+  for (int i = threadIdx.x; i < (t1 - t0) * p.half; i += CA_NT) {
+    const int tt = i / p.half, f = i - tt * p.half;
+    float sn, cs;
+    sincosf((float)p.positions[t0 + tt] * p.inv_freq[f], &sn, &cs);
+    s_cs[2 * i] = cs * p.rot_mult;
+    s_cs[2 * i + 1] = sn * p.rot_mult;
+  }
+  __syncthreads();
+  const int K = p.taps, hist_n = K - 1;
+  const int nq = p.H * p.M, nk = p.G * p.M;
+  const int C = (nq + nk) * p.D + p.G * p.Dv;
+  const T* w = reinterpret_cast<const T*>(p.w);
+  const int u_end = min(p.units, ((int)blockIdx.y + 1) * p.units_per_cta);
+  // both halves of a warp walk the same number of rounds; a half without a unit repeats the other's and stores nothing
+  for (int ub = blockIdx.y * p.units_per_cta + 2 * (threadIdx.x >> 5); ub < u_end; ub += CA_NT / 16) {
+    const bool mine = ub + (lane >> 4) < u_end;
+    const int u = mine ? ub + (lane >> 4) : ub;
+    const int kind = u < nq ? 0 : u < nq + nk ? 1 : 2;      // q, k, v
+    const int vh = kind == 2 ? (u - nq - nk) / p.vpieces : 0, vo = kind == 2 ? ((u - nq - nk) - vh * p.vpieces) * CA_VW : 0;      // value head, first column
+    const int n = kind == 2 ? min(CA_VW, p.Dv - vo) : p.D;
+    const int c0 = kind == 2 ? (nq + nk) * p.D + vh * p.Dv + vo : u * p.D;
+    const bool live = col < n;                              // n is a multiple of four: a lane's columns all count or none
+    const T* nw = reinterpret_cast<const T*>(kind == 0 ? p.qw : p.kw);
+    // taps right-aligned (slots below KM - K carry weight zero); the KM - 1 inputs before the group, then the group's rows
+    float wt[KM][4], seq[KM - 1 + AHEAD][4], nwv[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      nwv[i] = live ? ((kind < 2 && nw) ? ca_ld<T>(nw + col + i) : 1.f) : 0.f;
+#pragma unroll
+      for (int j = 0; j < KM; ++j) {
+        const int tap = j - (KM - K);
+        wt[j][i] = (tap >= 0 && live) ? ca_ld<T>(w + (size_t)(c0 + col + i) * K + tap) : 0.f;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < KM - 1 + AHEAD; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) seq[j][i] = 0.f;
+    const T* x = reinterpret_cast<const T*>(p.qkv) + c0 + col;
+    T* dst;                                                 // where token t0's (q) or slot 0's (k, v) columns go; lead: columns before the values
+    int width, lead = 0;
+    size_t step;
+    if (kind == 0) {
+      width = p.M * p.seg; lead = (u % p.M) * p.seg; step = (size_t)nq * width;
+      dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t0 * nq + u) * width;
+    } else if (kind == 1) {
+      width = p.seg; step = p.ldc;
+      dst = reinterpret_cast<T*>(p.kc) + (size_t)(u - nq) * p.seg;
+    } else {                                                // a head's last piece also writes the zeros behind the values
+      width = vo + CA_VW >= p.Dv ? p.wv - vo : n; step = p.ldc;
+      dst = reinterpret_cast<T*>(p.vc) + (size_t)vh * p.wv + vo;
+    }
+    const bool rot = kind < 2 && col < 2 * p.half;
+    const bool first = col < p.half;                        // half is a multiple of four: partners sit half / 4 lanes apart
+    const int partner = (lane & 16) | ((first ? hl + (p.half >> 2) : hl - (p.half >> 2)) & 15);
+    const float sg = first ? -1.f : 1.f;
+    int b = *s_b, bend = -1;                                // request at hand and its end (none yet)
+    for (int tg = t0; tg < t1; tg += AHEAD) {
+      if (live) {
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) ca_ld4(x + (size_t)min(tg + g, t1 - 1) * p.ld, seq[KM - 1 + g]);
+      }
+      float y[AHEAD][4];
+      if (min(tg + AHEAD, t1) <= bend) {                    // the whole group continues the request at hand
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < KM; ++j) acc += wt[j][i] * seq[g + j][i];
+            y[g][i] = acc;
+          }
+      } else {                                              // a request begins in the group: token by token, the inputs before it gathered anew
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) {
+          const int t = tg + g;
+          if (t < t1 && t >= bend) {
+            if (p.cu_q) {
+              while (b + 1 < p.B && t >= p.cu_q[b + 1]) ++b;          // tokens behind the last request (padded batches) count to it
+            } else {
+              b = t;
+            }
+            const int bq0 = p.cu_q ? p.cu_q[b] : b, bq1 = p.cu_q ? p.cu_q[b + 1] : b + 1;
+            bend = b + 1 < p.B ? bq1 : 0x7fffffff;
+            const bool fresh = p.seq_lens[b] - (bq1 - bq0) == 0;
+            const T* st = reinterpret_cast<const T*>(p.state) + ((size_t)p.req_slots[b] * C + c0 + col) * hist_n;
+#pragma unroll
+            for (int j = 0; j < KM - 1; ++j) {
+              const int tt = t - (KM - 1) + j;              // flat index of the input in slot j
+              if (j >= KM - K && live) {
+                if (tt >= bq0) {
+                  ca_ld4(x + (size_t)tt * p.ld, seq[g + j]);
+                } else {
+#pragma unroll
+                  for (int i = 0; i < 4; ++i) seq[g + j][i] = fresh ? 0.f : ca_ld<T>(st + (size_t)i * hist_n + (hist_n + tt - bq0));
+                }
+              }
+            }
+          }
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < KM; ++j) acc += wt[j][i] * seq[g + j][i];
+            y[g][i] = acc;
+          }
+          if (p.cu_q == nullptr && hist_n > 0 && t < t1 && live && mine) {
+            T* st = reinterpret_cast<T*>(p.state) + ((size_t)p.req_slots[b] * C + c0 + col) * hist_n;
+#pragma unroll
+            for (int j = 1; j < KM; ++j)
+              if (j >= KM - hist_n) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) ca_st<T>(st + (size_t)i * hist_n + (j - (KM - hist_n)), seq[g + j][i]);
+              }
+          }
+        }
+      }
+      if (p.qw) {                                           // unit RMS (the value units' sums go unused)
+        float ss[AHEAD];
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) ss[g] = y[g][0] * y[g][0] + y[g][1] * y[g][1] + y[g][2] * y[g][2] + y[g][3] * y[g][3];
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1)
+#pragma unroll
+          for (int g = 0; g < AHEAD; ++g) ss[g] += __shfl_xor_sync(0xffffffffu, ss[g], o);
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) {
+          const float r = kind < 2 ? 1.0f / sqrtf(ss[g] / (float)n + p.eps) : 1.f;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) y[g][i] *= r * nwv[i];
+        }
+      }
+      if (p.half > 0) {
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) {
+          float o[4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) o[i] = __shfl_sync(0xffffffffu, y[g][i], partner);
+          if (rot) {
+            const float* cs = s_cs + (size_t)min(tg + g - t0, t1 - t0 - 1) * p.half * 2 + 2 * (first ? col : col - p.half);
+            const float4 a = *reinterpret_cast<const float4*>(cs), c = *reinterpret_cast<const float4*>(cs + 4);          // cos, sin of four angles
+            y[g][0] = y[g][0] * a.x + sg * o[0] * a.y;
+            y[g][1] = y[g][1] * a.z + sg * o[1] * a.w;
+            y[g][2] = y[g][2] * c.x + sg * o[2] * c.y;
+            y[g][3] = y[g][3] * c.z + sg * o[3] * c.w;
+          }
+        }
+      }
+#pragma unroll
+      for (int g = 0; g < AHEAD; ++g) {
+        if (tg + g < t1 && mine) {
+          T* d = dst + (size_t)(kind == 0 ? tg + g - t0 : s_loc[tg + g - t0]) * step;
+          if (live) ca_st4(d + lead + col, y[g]);
+          const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+          for (int i = col; i < width; i += 64)
+            if (i < lead || i >= lead + n) ca_st4(d + i, zero);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < KM - 1; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) seq[j][i] = seq[j + AHEAD][i];
+    }
+  }
+}
+
 template <typename T, int EP, int KM>
 void launch_prep(const ConvPrepParams& p, bool vec, dim3 grid, size_t smem, cudaStream_t stream) {
   auto go = [&](auto kern) {
@@ -284,21 +489,37 @@ void conv_attention_prepare(const void* qkv, int ld, bool bf16, int T, int H, in
   p.positions = positions; p.cu_q = cu_q; p.req_slots = req_slots; p.seq_lens = seq_lens; p.B = B; p.qw = q_norm_w; p.kw = k_norm_w; p.eps = eps;
   p.inv_freq = inv_freq; p.half = inv_freq ? half : 0; p.rot_mult = rot_mult; p.kc = kc; p.vc = vc; p.ldc = ldc; p.loc = loc; p.q_out = q_out;
   p.seg = pad > 0 ? pad / M : D; p.wv = pad > 0 ? pad : Dv;
-  p.units = (H + G) * M + G;
-  // few tokens: one per CTA and the units spread over many CTAs; long batches: runs of tokens, all the history reads amortised
-  p.run = cu_q == nullptr ? 1 : T >= 4 * num_sms ? 16 : 4;
-  const int cols = (T + p.run - 1) / p.run;
-  int ys = std::max(1, std::min((p.units + 7) / 8, (4 * num_sms + cols - 1) / cols));
-  p.units_per_cta = ((p.units + ys - 1) / ys + 7) / 8 * 8;
-  ys = (p.units + p.units_per_cta - 1) / p.units_per_cta;
-  const int n = std::max(D, Dv), ep = n <= 64 ? 1 : n <= 128 ? 2 : 4;
-  const size_t smem = sizeof(float) * ((size_t)p.run * p.half * 2 + 8 * 64 * ep) + sizeof(int) * 4;
   const size_t a2 = bf16 ? 4 : 8;
-  auto al = [&](const void* q) { return ((uintptr_t)q % a2) == 0; };
-  const bool vec = D % 2 == 0 && Dv % 2 == 0 && ld % 2 == 0 && ldc % 2 == 0 && p.seg % 2 == 0 && p.wv % 2 == 0 && al(qkv) && al(kc) && al(vc) && al(q_out);
+  auto al = [&](const void* q, size_t n) { return ((uintptr_t)q % n) == 0; };
+  auto even = [&](int k) {                                  // every width and stride a multiple of k elements, every base aligned to as much
+    const size_t n = a2 * k / 2;
+    return D % k == 0 && Dv % k == 0 && ld % k == 0 && ldc % k == 0 && p.seg % k == 0 && p.wv % k == 0 && al(qkv, n) && al(kc, n) && al(vc, n) && al(q_out, n);
+  };
+  const bool x4 = D <= 64 && taps <= 4 && p.half % 4 == 0 && even(4);
+  p.vpieces = x4 ? (Dv + CA_VW - 1) / CA_VW : 1;
+  p.units = (H + G) * M + G * p.vpieces;
+  // few tokens: one per CTA and the units spread over many CTAs; long batches: runs of tokens, all the history reads amortised
+  p.run = cu_q == nullptr ? 1 : T >= 16 * num_sms ? 32 : T >= 4 * num_sms ? 16 : 4;
+  const int cols = (T + p.run - 1) / p.run, step = x4 ? 16 : 8;          // units a CTA walks at once
+  int ys = std::max(1, std::min((p.units + step - 1) / step, (4 * num_sms + cols - 1) / cols));
+  p.units_per_cta = ((p.units + ys - 1) / ys + step - 1) / step * step;
+  ys = (p.units + p.units_per_cta - 1) / p.units_per_cta;
   dim3 grid(cols, ys);
-  if (bf16) dispatch_prep<__nv_bfloat16>(p, vec, grid, smem, stream);
-  else dispatch_prep<float>(p, vec, grid, smem, stream);
+  if (x4) {
+    const size_t smem = sizeof(float) * (size_t)p.run * p.half * 2 + sizeof(int) * (p.run + 4);      // at most 17 KB
+    if (cu_q == nullptr) {
+      if (bf16) conv_attention_prepare_x4_kernel<__nv_bfloat16, 1><<<grid, CA_NT, smem, stream>>>(p);
+      else conv_attention_prepare_x4_kernel<float, 1><<<grid, CA_NT, smem, stream>>>(p);
+    } else {
+      if (bf16) conv_attention_prepare_x4_kernel<__nv_bfloat16, 4><<<grid, CA_NT, smem, stream>>>(p);
+      else conv_attention_prepare_x4_kernel<float, 4><<<grid, CA_NT, smem, stream>>>(p);
+    }
+  } else {
+    const int n = std::max(D, Dv), ep = n <= 64 ? 1 : n <= 128 ? 2 : 4;
+    const size_t smem = sizeof(float) * ((size_t)p.run * p.half * 2 + 8 * 64 * ep) + sizeof(int) * 4;
+    if (bf16) dispatch_prep<__nv_bfloat16>(p, even(2), grid, smem, stream);
+    else dispatch_prep<float>(p, even(2), grid, smem, stream);
+  }
   SGLB_CUDA_CHECK(cudaGetLastError());
   if (cu_q != nullptr) causal_conv1d_state(qkv, ld, conv_state, cu_q, req_slots, seq_lens, B, (H + G) * M * D + G * Dv, taps, bf16, stream);
 }

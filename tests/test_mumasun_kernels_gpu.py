@@ -98,7 +98,7 @@ def test_experts_with_weighted_inputs(T, W, I, E, K, dtype):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("H,G,M,D,Dv,rot,taps,pad", [(4, 2, 2, 64, 128, 64, 3, 0), (4, 2, 2, 64, 128, 64, 3, 128), (6, 3, 2, 24, 40, 16, 2, 128), (3, 1, 2, 7, 9, 6, 5, 0),
-                                                     (2, 2, 2, 130, 200, 20, 4, 0), (2, 1, 1, 16, 16, 0, 1, 0), (4, 4, 2, 33, 65, 0, 16, 0), (2, 1, 1, 100, 96, 100, 4, 128)])
+                                                     (2, 2, 2, 130, 200, 20, 4, 0), (2, 1, 1, 16, 16, 0, 1, 0), (4, 4, 2, 33, 65, 0, 16, 0), (2, 1, 1, 100, 96, 100, 4, 128), (2, 1, 2, 12, 72, 8, 4, 0), (3, 1, 1, 64, 100, 64, 1, 0), (5, 5, 2, 4, 4, 0, 4, 0)])
 def test_conv_attention_prepare(H, G, M, D, Dv, rot, taps, pad, dtype):
     """ragged portions (single tokens among them, cached history, empty requests), then decode steps of all requests: q rows, cache rows and state"""
     _need()
@@ -140,6 +140,33 @@ def test_conv_attention_prepare(H, G, M, D, Dv, rot, taps, pad, dtype):
         torch.testing.assert_close(v1.cpu().float(), v0.float(), **t)
         if taps > 1:
             assert torch.equal(st1.cpu(), st0), n_step                        # the state holds projections: moved, never computed
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("lens", [[2700], [1, 900, 3, 0, 1501, 40, 2, 310], [5] * 520])
+def test_conv_attention_prepare_long_batches(lens, dtype):
+    """long runs of tokens per CTA: requests that begin and end inside a run and inside a group of four rows"""
+    _need()
+    g = torch.Generator().manual_seed(len(lens))
+    H, G, D, Dv, rot, taps, B, T = 2, 1, 8, 12, 8, 4, len(lens), sum(lens)
+    C = 2 * (H + G) * D + G * Dv
+    x, w = torch.randn(T, C, generator=g).to(dtype), (torch.randn(C, taps, generator=g) * 0.5).to(dtype)
+    st0 = torch.randn(B + 1, C, taps - 1, generator=g).to(dtype)
+    st1, f = st0.to(DEV), yarn_inv_freq(rot, 500.0)[0]
+    cached = [(3 * i) % 5 for i in range(B)]
+    pos = _i32([c + i for c, n in zip(cached, lens) for i in range(n)], "cpu")
+    k0 = [torch.zeros(T + 3, 1, 16, dtype=dtype) for _ in range(2)]
+    k1 = [t.to(DEV) for t in k0]
+    loc = torch.randperm(T, generator=g).int() + 3
+    cu, sl, slots = _i32(np.concatenate([[0], np.cumsum(lens)]).tolist(), "cpu"), _i32([a + b for a, b in zip(lens, cached)], "cpu"), torch.randperm(B, generator=g).int() + 1
+    nq, nk = (torch.rand(D, generator=g) + 0.5).to(dtype), (torch.rand(D, generator=g) + 0.5).to(dtype)
+    q0 = torch_ref.conv_attention_prepare(x, H, G, 2, D, Dv, w, st0, pos, cu, slots, sl, nq, nk, 1e-5, f, 1.1, *k0, loc)
+    c = lambda t: t.to(DEV)
+    q1 = ops.conv_attention_prepare(c(x), H, G, 2, D, Dv, c(w), st1, c(pos), c(cu), c(slots), c(sl), c(nq), c(nk), 1e-5, c(f), 1.1, *k1, c(loc))
+    t = _tol(dtype, f32=(1e-3, 1e-3), bf=(1e-2, 1e-2))
+    for a, b in ((q1, q0), (k1[0], k0[0]), (k1[1], k0[1])):
+        torch.testing.assert_close(a.cpu().float(), b.float(), **t)
+    assert torch.equal(st1.cpu(), st0)
 
 
 def _attention_case(H, G, D, Dv, lens, cached, ps, chunk, dtype, tc, seed=0, decode=False, splits=1):
