@@ -168,7 +168,7 @@ def check_chunk_edges(device, dtype, ps, D, Dv, tol, tc_route=True):
     """one key stands out for one query; just inside the query's chunk its value takes over, just outside it is not seen.  Keys at the chunk's first
     position, at page borders and far back among hundreds; the query in a prompt, at the start of a portion, and decoded alone"""
     H, G = 2, 1
-    for chunk, i, j in ((16, 31, 16), (16, 32, 31), (16, 31, 15), (120, 119, 0), (120, 120, 119), (120, 239, 120), (120, 239, 119), (0, 299, 3), (300, 299, 0), (300, 300, 299),
+    for chunk, i, j in ((16, 31, 16), (16, 32, 31), (16, 31, 15), (110, 109, 0), (110, 110, 109), (110, 219, 110), (110, 219, 109), (0, 299, 3), (300, 299, 0), (300, 300, 299),
                         (13, 25, 13), (13, 26, 25), (64, 127, 64), (64, 128, 127), (1, 5, 4), (1, 5, 5), (7, 48, 42), (7, 49, 48)):
         if j > i:
             continue
