@@ -458,9 +458,28 @@ def mumasun_config(hf: Dict[str, Any]) -> Dict[str, Any]:
                 hybrid={"layers": layers, "logit_scale": float(1.0 if hf.get("logit_scale") is None else hf["logit_scale"])})
 
 
+def surasun_config(hf: Dict[str, Any]) -> Dict[str, Any]:
+    """Surasun ``config.json`` -> ModelConfig fields.  ``layers[i]`` = ``type`` of the mixer (``mamba2`` | ``parallel`` | ``rglru``), its sizes and constants
+    under ``mixer`` (a parallel mixer: ``left`` / ``right`` with ``left_scale`` / ``right_scale``), the feed-forward under ``mlp`` (``kind`` ``dense``) or
+    null; ``streams`` and ``residual_mult`` of the hyper-connections; globals ``width``, ``vocab``, ``norm.eps``.  The flat fields are summaries
+    for code that sizes buffers; the model reads ``hybrid``."""
+    layers = [dict(l) for l in hf["layers"]]
+    width = int(hf["width"])
+    attn = [l["mixer"]["left"] for l in layers if l["type"] == "parallel"]
+    heads = max([int(m["heads"]) for m in attn] or [1])
+    return dict(architecture="Surasun", hidden_size=width, vocab_size=int(hf["vocab"]), num_hidden_layers=len(layers),
+                rms_norm_eps=float((hf.get("norm") or {}).get("eps", 1e-5)), final_logit_softcapping=0.0,
+                num_attention_heads=heads, num_key_value_heads=1, head_dim=max([int(m["dim"]) for m in attn] or [width // heads]),
+                intermediate_size=max([int(l["mlp"]["ff"]) for l in layers if l.get("mlp")] or [width]), num_local_experts=0, num_experts_per_tok=0,
+                max_position_embeddings=int(hf.get("max_positions") or (1 << 20)), tie_word_embeddings=True, eos_token_id=None,
+                dtype={"float16": "float16", "float32": "float32"}.get(hf.get("dtype") or "bfloat16", "bfloat16"),
+                hybrid={"layers": layers, "streams": int(hf.get("streams") or 1),
+                        "residual_mult": float(1.0 if hf.get("residual_mult") is None else hf["residual_mult"])})
+
+
 # configurations that list their layers one by one, chosen by the file's ``architecture`` key
 _LAYER_LIST_READERS = {"Rirotar": rirotar_config, "Zaparax": zaparax_config, "Resatar": resatar_config, "Rumuvik": rumuvik_config,
-                       "Mumasun": mumasun_config}
+                       "Mumasun": mumasun_config, "Surasun": surasun_config}
 
 
 def _has_native_class(arch: str) -> bool:

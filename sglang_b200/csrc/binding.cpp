@@ -201,13 +201,13 @@ void causal_conv1d(const at::Tensor& x, const at::Tensor& w, c10::optional<at::T
   TORCH_CHECK((bf16 || x.scalar_type() == at::kFloat) && w.scalar_type() == x.scalar_type() && conv_state.scalar_type() == x.scalar_type(),
               "causal_conv1d: x / weight / state must share bf16 or fp32");
   const int C = (int)x.size(1), K = (int)w.size(1);
-  TORCH_CHECK(w.size(0) == C && conv_state.size(1) == C && conv_state.size(2) == K - 1 && u.scalar_type() == at::kFloat && u.stride(1) == 1 &&
-              u.size(0) == x.size(0) && u.size(1) == C);
+  TORCH_CHECK(w.size(0) == C && conv_state.size(1) == C && conv_state.size(2) == K - 1 && (u.scalar_type() == at::kFloat || u.scalar_type() == x.scalar_type()) &&
+              u.stride(1) == 1 && u.size(0) == x.size(0) && u.size(1) == C);
   if (bias.has_value()) TORCH_CHECK(bias->scalar_type() == x.scalar_type() && bias->numel() == C);
   c10::cuda::CUDAGuard g(x.device());
   sglb::causal_conv1d(x.data_ptr(), (int)x.stride(0), w.data_ptr(), bias.has_value() ? bias->data_ptr() : nullptr, conv_state.data_ptr(),
                       opt_ptr<int>(cu_q), req_slots.data_ptr<int>(), seq_lens.data_ptr<int>(), (int)req_slots.size(0), (int)max_q_len, C, K, silu, bf16,
-                      u.data_ptr<float>(), (int)u.stride(0), cur_stream());
+                      u.data_ptr(), u.scalar_type() == at::kBFloat16, (int)u.stride(0), cur_stream());
   count(2);
 }
 
@@ -342,18 +342,100 @@ void postnorm_add_rmsnorm_f32(at::Tensor residual, const at::Tensor& delta, cons
   count();
 }
 
-void grouped_rmsnorm(const at::Tensor& x, const at::Tensor& w, int64_t groups, double eps, at::Tensor out, c10::optional<at::Tensor> gate, double out_scale) {
+void grouped_rmsnorm(const at::Tensor& x, c10::optional<at::Tensor> w, int64_t groups, double eps, at::Tensor out, c10::optional<at::Tensor> gate,
+                     double out_scale, bool silu) {
   CHECK_CUDA(x);
-  TORCH_CHECK(x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous() && out.dim() == 2 && out.stride(1) == 1 && w.is_contiguous() &&
-              bf16_or_f32(out) && out.scalar_type() == w.scalar_type() && out.size(0) == x.size(0) && out.size(1) == x.size(1) && w.numel() == x.size(1));
+  TORCH_CHECK(x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous() && out.dim() == 2 && out.stride(1) == 1 && bf16_or_f32(out) &&
+              out.size(0) == x.size(0) && out.size(1) == x.size(1));
+  if (w.has_value()) TORCH_CHECK(w->is_contiguous() && out.scalar_type() == w->scalar_type() && w->numel() == x.size(1));
   if (gate.has_value())
     TORCH_CHECK(gate->scalar_type() == out.scalar_type() && gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == x.size(0) &&
                 gate->size(1) == x.size(1));
   if (x.size(0) == 0) return;
   c10::cuda::CUDAGuard g(x.device());
-  sglb::grouped_rmsnorm(x.data_ptr<float>(), w.data_ptr(), out.data_ptr(), out.scalar_type() == at::kBFloat16, (int)x.size(0), (int)x.size(1), (int)groups,
-                        (float)eps, gate.has_value() ? gate->data_ptr() : nullptr, gate.has_value() ? (int)gate->stride(0) : 0, (int)out.stride(0),
-                        (float)out_scale, cur_stream());
+  sglb::grouped_rmsnorm(x.data_ptr<float>(), w.has_value() ? w->data_ptr() : nullptr, out.data_ptr(), out.scalar_type() == at::kBFloat16, (int)x.size(0),
+                        (int)x.size(1), (int)groups, (float)eps, gate.has_value() ? gate->data_ptr() : nullptr, gate.has_value() ? (int)gate->stride(0) : 0,
+                        (int)out.stride(0), (float)out_scale, silu, cur_stream());
+  count();
+}
+
+void stream_mix_norm(c10::optional<at::Tensor> x, c10::optional<at::Tensor> table, c10::optional<at::Tensor> ids, c10::optional<at::Tensor> y,
+                     const at::Tensor& coef, int64_t S, const at::Tensor& w, double eps, bool centre, c10::optional<at::Tensor> xn, at::Tensor h) {
+  CHECK_CUDA(h);
+  const int64_t T = h.size(0), W = h.size(1);
+  const auto dt = h.scalar_type();
+  TORCH_CHECK(bf16_or_f32(h) && h.dim() == 2 && h.is_contiguous() && w.is_contiguous() && w.scalar_type() == dt && w.numel() == W && S >= 1 &&
+              coef.is_cuda() && coef.scalar_type() == at::kFloat && coef.is_contiguous() && coef.numel() == S * S + 2 * S);
+  TORCH_CHECK(x.has_value() != (table.has_value() && ids.has_value()), "stream_mix_norm: either the streams or an embedding table with ids");
+  auto streams_ok = [&](const at::Tensor& t) {
+    return t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.dim() == 3 && t.size(0) == T && t.size(1) == S && t.size(2) == W;
+  };
+  if (x.has_value()) {
+    TORCH_CHECK(streams_ok(*x));
+  } else {
+    CHECK_I32(*ids);
+    TORCH_CHECK(table->is_cuda() && table->scalar_type() == dt && table->is_contiguous() && table->dim() == 2 && table->size(1) == W && table->size(0) >= 1 &&
+                ids->is_contiguous() && ids->numel() == T);
+  }
+  if (xn.has_value()) TORCH_CHECK(streams_ok(*xn));
+  if (y.has_value()) TORCH_CHECK(y->is_cuda() && y->scalar_type() == dt && y->is_contiguous() && y->numel() == T * W);
+  if (T == 0) return;
+  c10::cuda::CUDAGuard g(h.device());
+  sglb::stream_mix_norm(opt_ptr<float>(x), x.has_value() ? nullptr : table->data_ptr(), x.has_value() ? nullptr : ids->data_ptr<int>(),
+                        x.has_value() ? 0 : (int)table->size(0), y.has_value() ? y->data_ptr() : nullptr, coef.data_ptr<float>(), (int)S, w.data_ptr(),
+                        xn.has_value() ? xn->data_ptr<float>() : nullptr, h.data_ptr(), dt == at::kBFloat16, (int)T, (int)W, (float)eps, centre, cur_stream());
+  count();
+}
+
+void linear_attention_prepare(const at::Tensor& proj, int64_t H, int64_t D, int64_t Dv, const at::Tensor& positions, c10::optional<at::Tensor> inv_freq,
+                              bool interleaved, double k_scale, bool silu, at::Tensor u) {
+  CHECK_CUDA(proj); CHECK_I32(positions);
+  const int64_t T = proj.size(0);
+  TORCH_CHECK(bf16_or_f32(proj) && proj.dim() == 2 && proj.stride(1) == 1 && proj.size(1) >= H * (Dv + 2 * D) && positions.numel() == T &&
+              u.scalar_type() == at::kFloat && u.is_contiguous() && u.dim() == 2 && u.size(0) == T && u.size(1) == H * (Dv + 2 * D));
+  int half = 0;
+  if (inv_freq.has_value()) {
+    TORCH_CHECK(inv_freq->is_cuda() && inv_freq->scalar_type() == at::kFloat && inv_freq->is_contiguous() && 2 * inv_freq->numel() <= D);
+    half = (int)inv_freq->numel();
+  }
+  if (T == 0) return;
+  c10::cuda::CUDAGuard g(proj.device());
+  sglb::linear_attention_prepare(proj.data_ptr(), (int)proj.stride(0), proj.scalar_type() == at::kBFloat16, (int)T, (int)H, (int)D, (int)Dv,
+                                 positions.data_ptr<int>(), half > 0 ? inv_freq->data_ptr<float>() : nullptr, half, interleaved, (float)k_scale, silu,
+                                 u.data_ptr<float>(), cur_stream());
+  count();
+}
+
+// u [T, blocks * n] x w [blocks, rows, n] -> fp32 [T, blocks, rows]
+void gemm_diag_f32(const at::Tensor& u, const at::Tensor& w, at::Tensor out) {
+  CHECK_CUDA(u); CHECK_BF16(u); CHECK_BF16(w);
+  TORCH_CHECK(u.dim() == 2 && u.stride(1) == 1 && w.dim() == 3 && w.is_contiguous() && u.size(1) == w.size(0) * w.size(2) && out.scalar_type() == at::kFloat &&
+              out.is_contiguous() && out.numel() == u.size(0) * w.size(0) * w.size(1));
+  TORCH_CHECK(((uintptr_t)u.data_ptr() & 15) == 0 && ((uintptr_t)w.data_ptr() & 15) == 0 && ((uintptr_t)out.data_ptr() & 15) == 0);
+  if (u.size(0) == 0) return;
+  c10::cuda::CUDAGuard g(u.device());
+  sglb::gemm_bf16_tc_diag_f32(u.data_ptr(), w.data_ptr(), out.data_ptr<float>(), (int)u.size(0), (int)w.size(0), (int)w.size(1), (int)w.size(2), (int)u.stride(0),
+                              num_sms(), cur_stream());
+  count();
+}
+
+void rglru_scan(const at::Tensor& gates, c10::optional<at::Tensor> bias, const at::Tensor& u, const at::Tensor& lam, const at::Tensor& y, at::Tensor state,
+                const at::Tensor& req_slots, const at::Tensor& seq_lens, c10::optional<at::Tensor> cu_q, int64_t blocks, double power, at::Tensor out) {
+  CHECK_CUDA(gates); CHECK_I32(req_slots); CHECK_I32(seq_lens);
+  const int64_t T = u.size(0), C = u.size(1);
+  auto f32c = [](const at::Tensor& t) { return t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous(); };
+  TORCH_CHECK(f32c(gates) && gates.numel() == T * 2 * C && f32c(lam) && lam.numel() == C && f32c(state) && state.numel() == state.size(0) * C && blocks >= 1 &&
+              C % blocks == 0);
+  TORCH_CHECK(bf16_or_f32(u) && u.dim() == 2 && u.stride(1) == 1 && y.dim() == 2 && y.stride(1) == 1 && y.scalar_type() == u.scalar_type() && y.size(0) == T &&
+              y.size(1) == C && out.scalar_type() == u.scalar_type() && out.is_contiguous() && out.numel() == T * C);
+  if (bias.has_value()) TORCH_CHECK(f32c(*bias) && bias->numel() == 2 * C);
+  const int B = (int)req_slots.size(0);
+  if (cu_q.has_value()) { CHECK_I32(*cu_q); TORCH_CHECK(cu_q->numel() == B + 1); } else TORCH_CHECK(T == B);
+  if (T == 0) return;
+  c10::cuda::CUDAGuard g(u.device());
+  sglb::rglru_scan(gates.data_ptr<float>(), opt_ptr<float>(bias), u.data_ptr(), (int)u.stride(0), lam.data_ptr<float>(), y.data_ptr(), (int)y.stride(0),
+                   u.scalar_type() == at::kBFloat16, state.data_ptr<float>(), req_slots.data_ptr<int>(), seq_lens.data_ptr<int>(), opt_ptr<int>(cu_q), B, (int)C,
+                   (int)blocks, (float)power, out.data_ptr(), cur_stream());
   count();
 }
 
@@ -547,7 +629,7 @@ void mamba1_scan(const at::Tensor& u, const at::Tensor& dt_raw, c10::optional<at
 void attention_prepare(const at::Tensor& qkv, int64_t H, int64_t G, int64_t D, int64_t Dv, const at::Tensor& positions, at::Tensor k_cache, at::Tensor v_cache,
                        const at::Tensor& loc, c10::optional<at::Tensor> q_norm_w, c10::optional<at::Tensor> k_norm_w, double eps,
                        c10::optional<at::Tensor> inv_freq, c10::optional<at::Tensor> v_first, double v_lambda, at::Tensor q_out, int64_t pad,
-                       c10::optional<at::Tensor> v_inv_freq, bool v_interleaved) {
+                       c10::optional<at::Tensor> v_inv_freq, bool v_interleaved, bool interleaved) {
   CHECK_CUDA(qkv); CHECK_I32(positions); CHECK_I32(loc);
   const int64_t T = qkv.size(0);
   TORCH_CHECK(bf16_or_f32(qkv) && qkv.dim() == 2 && qkv.stride(1) == 1 && qkv.size(1) >= H * D + G * D + G * Dv && H % G == 0);
@@ -577,7 +659,7 @@ void attention_prepare(const at::Tensor& qkv, int64_t H, int64_t G, int64_t D, i
                           positions.data_ptr<int>(), q_norm_w.has_value() ? q_norm_w->data_ptr() : nullptr, k_norm_w.has_value() ? k_norm_w->data_ptr() : nullptr,
                           (float)eps, half > 0 ? inv_freq->data_ptr<float>() : nullptr, half, v_first.has_value() ? v_first->data_ptr() : nullptr,
                           v_first.has_value() ? (int)v_first->stride(0) : 0, (float)v_lambda, k_cache.data_ptr(), v_cache.data_ptr(), (size_t)k_cache.stride(0),
-                          loc.data_ptr<int>(), q_out.data_ptr(), (int)pad, opt_ptr<float>(v_inv_freq), v_interleaved, cur_stream());
+                          loc.data_ptr<int>(), q_out.data_ptr(), (int)pad, opt_ptr<float>(v_inv_freq), v_interleaved, interleaved, cur_stream());
   count();
 }
 
@@ -1235,14 +1317,22 @@ TORCH_LIBRARY(sglb, m) {
         "int max_q_len, float scale, int mul_prev, int mul_cur, int buckets, Tensor(b!) out) -> ()", &bigram_embedding);
   m.def("postnorm_add_rmsnorm_f32(Tensor(a!) residual, Tensor delta, Tensor post_w, Tensor w, Tensor(b!) out, float eps, bool zero_centred=True) -> ()",
         &postnorm_add_rmsnorm_f32);
-  m.def("grouped_rmsnorm(Tensor x, Tensor w, int groups, float eps, Tensor(a!) out, Tensor? gate=None, float out_scale=1.0) -> ()", &grouped_rmsnorm);
+  m.def("grouped_rmsnorm(Tensor x, Tensor? w, int groups, float eps, Tensor(a!) out, Tensor? gate=None, float out_scale=1.0, bool silu=False) -> ()",
+        &grouped_rmsnorm);
+  m.def("stream_mix_norm(Tensor? x, Tensor? table, Tensor? ids, Tensor? y, Tensor coef, int streams, Tensor w, float eps, bool centre, Tensor(a!)? xn, "
+        "Tensor(b!) h) -> ()", &stream_mix_norm);
+  m.def("linear_attention_prepare(Tensor proj, int H, int D, int Dv, Tensor positions, Tensor? inv_freq, bool interleaved, float k_scale, bool silu, "
+        "Tensor(a!) u) -> ()", &linear_attention_prepare);
+  m.def("gemm_diag_f32(Tensor u, Tensor w, Tensor(a!) out) -> ()", &gemm_diag_f32);
+  m.def("rglru_scan(Tensor gates, Tensor? bias, Tensor u, Tensor lam, Tensor y, Tensor(a!) state, Tensor req_slots, Tensor seq_lens, Tensor? cu_q, int blocks, "
+        "float power, Tensor(b!) out) -> ()", &rglru_scan);
   m.def("mamba2_scan(Tensor u, Tensor? z, Tensor? dt_raw, Tensor? dt_bias, Tensor? A_log, Tensor? D, Tensor(a!) state, Tensor req_slots, Tensor seq_lens, "
         "Tensor? cu_q, int H, int P, int N, int G, Tensor(b!) out, Tensor? decay=None, Tensor? gates=None) -> ()", &mamba2_scan);
   m.def("mamba1_scan(Tensor u, Tensor dt_raw, Tensor? dt_bias, Tensor A_log, Tensor Bm, Tensor Cm, Tensor? D, Tensor? z, Tensor(a!) state, Tensor req_slots, "
         "Tensor seq_lens, Tensor? cu_q, Tensor(b!) out) -> ()", &mamba1_scan);
   m.def("attention_prepare(Tensor qkv, int H, int G, int D, int Dv, Tensor positions, Tensor(a!) k_cache, Tensor(b!) v_cache, Tensor loc, Tensor? q_norm_w, "
         "Tensor? k_norm_w, float eps, Tensor? inv_freq, Tensor? v_first, float v_lambda, Tensor(c!) q_out, int pad=0, Tensor? v_inv_freq=None, "
-        "bool v_interleaved=False) -> ()", &attention_prepare);
+        "bool v_interleaved=False, bool interleaved=False) -> ()", &attention_prepare);
   m.def("sigmoid_gate(Tensor o, Tensor gate, int Dv, float out_scale, Tensor(a!) out) -> ()", &sigmoid_gate);
   m.def("activation(Tensor x, int act, Tensor(a!) out, Tensor? mul=None) -> ()", &activation);
   m.def("qk_norm_cache_write(Tensor qkv, int H, int G, int D, int Dv, Tensor positions, float eps, float temp_coef, int temp_every, "

@@ -48,6 +48,7 @@ void attn_fwd_tc(const void* q, const void* k_cache, const void* v_cache, void* 
 void gemm_bf16_tc(const void* A, const void* W, void* C, const void* bias, int M, int N, int K, int lda, int ldw, int ldc,
                   int epilogue, int bn, int num_sms, cudaStream_t stream);
 int gemm_pick_bn(int M, int N, int K, int num_sms);
+void gemm_bf16_tc_diag_f32(const void* A, const void* W, float* C, int M, int blocks, int rows, int K, int lda, int num_sms, cudaStream_t stream);
 void gemm_bf16_tc_grouped(const void* A, const void* W, void* C, const float* row_scale, int M_cap, int n_out, int K, int lda,
                           int ldc, int num_experts, const int* tile_expert, const int* num_m_tiles, bool split_silu, int num_sms,
                           cudaStream_t stream, bool relu2 = false);
@@ -101,7 +102,8 @@ void sample(const void* logits, bool bf16, int B, int V, int stride, const float
 void causal_conv1d_state(const void* x, int ldx, void* conv_state, const int* cu_q, const int* req_slots, const int* seq_lens, int B, int C, int K,
                          bool bf16, cudaStream_t stream);
 void causal_conv1d(const void* x, int ldx, const void* w, const void* bias, void* conv_state, const int* cu_q, const int* req_slots,
-                   const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, float* u, int ldu, cudaStream_t stream);
+                   const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, void* u, bool u_bf16, int ldu,
+                   cudaStream_t stream);
 void selective_state_update(float* state, const int* req_slots, const float* x, int ldx, const float* dt, const float* A, const float* Bm,
                             const float* Cm, int ldbc, const float* Dv, int B, int H, int P, int N, int G, float* y, cudaStream_t stream);
 bool gated_delta_update(float* state, const int* req_slots, const float* u, int ldu, int k_off, int v_off, const float* g, const float* beta, int B,
@@ -125,7 +127,7 @@ void sigmoid_gate(const void* o, int head_stride, const void* gate, int ldg, boo
                   cudaStream_t stream);
 void attention_prepare(const void* qkv, int ld, bool bf16, int T, int H, int G, int D, int Dv, const int* positions, const void* q_norm_w, const void* k_norm_w,
                        float eps, const float* inv_freq, int half, const void* v_first, int ldvf, float lam, void* kc, void* vc, size_t ldc, const int* loc,
-                       void* q_out, int pad, const float* v_inv_freq, bool v_interleaved, cudaStream_t stream);
+                       void* q_out, int pad, const float* v_inv_freq, bool v_interleaved, bool interleaved, cudaStream_t stream);
 void rotate_heads(const void* o, int head_stride, bool bf16, const int* positions, const float* inv_freq, int T, int H, int Dv, bool interleaved, bool inverse,
                   const float* lse, const float* sinks, void* out, cudaStream_t stream);
 void causal_softmax(const float* scores, void* out, bool out_bf16, int rows, int tq, int n, int first, float scale, cudaStream_t stream);
@@ -149,7 +151,14 @@ void norm_add_f32(float* x, const void* src, bool src_bf16, const int* ids, int 
 void parallel_add_rmsnorm_f32(float* residual, const void* d1, const void* d2, bool delta_bf16, const float* d3, const void* w1, const void* w2, void* out1,
                               void* out2, bool out_bf16, int T, int H, float eps, bool zero_centred, cudaStream_t stream);
 void grouped_rmsnorm(const float* x, const void* w, void* out, bool out_bf16, int T, int C, int groups, float eps, const void* gate, int ldg, int ldo,
-                     float out_scale, cudaStream_t stream);
+                     float out_scale, bool silu, cudaStream_t stream);
+void stream_mix_norm(const float* x, const void* table, const int* ids, int rows, const void* y, const float* coef, int streams, const void* w, float* xn,
+                     void* h, bool bf16, int T, int W, float eps, bool centre, cudaStream_t stream);
+void linear_attention_prepare(const void* proj, int ld, bool bf16, int T, int H, int D, int Dv, const int* positions, const float* inv_freq, int half,
+                              bool interleaved, float k_scale, bool silu, float* u, cudaStream_t stream);
+// rglru.cu
+void rglru_scan(const float* gates, const float* bias, const void* u, int ldu, const float* lam, const void* y, int ldy, bool bf16, float* state,
+                const int* req_slots, const int* seq_lens, const int* cu_q, int B, int C, int blocks, float power, void* out, cudaStream_t stream);
 void bigram_embedding(const void* embed, const void* bigram, bool bf16, const int* ids, int* prev_tokens, const int* cu_q, const int* req_slots,
                       const int* seq_lens, int B, int max_q_len, int W, int vocab, float scale, long long mul_prev, long long mul_cur, int buckets,
                       float* out, cudaStream_t stream);

@@ -19,12 +19,16 @@ constexpr int GEMM_BM = 128;
 constexpr int GEMM_BK = 64;
 constexpr int GEMM_THREADS = 256;
 
-enum GemmEpilogue { EPI_NONE = 0, EPI_BIAS = 1, EPI_SILU_MUL = 2, EPI_PUSH = 3, EPI_SILU_SPLIT = 4, EPI_ROWSCALE = 5, EPI_RELU2 = 6 };
+enum GemmEpilogue { EPI_NONE = 0, EPI_BIAS = 1, EPI_SILU_MUL = 2, EPI_PUSH = 3, EPI_SILU_SPLIT = 4, EPI_ROWSCALE = 5, EPI_RELU2 = 6,
+                    EPI_F32_DIAG = 7 };
 // EPI_SILU_SPLIT: W = [gate rows (n_half) ; up rows (n_half)] un-interleaved (the checkpoint layout).  Each B stage is
 //   filled by TWO TMA boxes of BN/2 rows — gate rows j.. and up rows n_half+j.. — so one UMMA of width BN produces the
 //   gate half in accumulator columns [0,BN/2) and the matching up half in [BN/2,BN); the epilogue writes silu(g)*u.
 // EPI_RELU2    : C = max(acc, 0)^2 (ungated experts).
 // EPI_ROWSCALE : C[row,:] = acc[row,:] * scale[row]  (fp32 per-row scale passed through `bias`; MoE routing weights).
+// EPI_F32_DIAG : block-diagonal W with an fp32 result: row block j of W (n_half rows; tiles do not straddle blocks) multiplies columns
+//   [j*K, (j+1)*K) of A, so that C[:, j*n_half ..] = A_j W_j^T in fp32 (C points to floats, ldc counts floats).  A K step that reaches beyond
+//   column K of its block reads zeros from W's tensor map.
 // GROUPED      : A rows are expert-sorted and padded to 128-row tiles; W is [E][N][K] behind a 3-D tensor map and
 //   tile_expert[m_tile] selects the expert slab; the number of live M tiles is read from device memory.
 
@@ -102,10 +106,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x) {
       const int m_blk = tile % m_tiles, n_blk = tile / m_tiles;
       const int expert = GROUPED ? __ldg(tile_expert + m_blk) : 0;
+      const int a_col = EPI == EPI_F32_DIAG ? (n_blk * BN / n_half) * K : 0;
       for (int kb = 0; kb < num_kb; ++kb) {
         mbar_wait(&empty[stage], phase ^ 1);
         mbar_expect_tx(&full[stage], Cfg::STAGE_BYTES);
-        tma_load_2d(sA + stage * Cfg::A_BYTES, &tmA, &full[stage], kb * GEMM_BK, m_blk * GEMM_BM);
+        tma_load_2d(sA + stage * Cfg::A_BYTES, &tmA, &full[stage], a_col + kb * GEMM_BK, m_blk * GEMM_BM);
         uint8_t* b_dst = sB + stage * Cfg::B_BYTES;
         if constexpr (GROUPED) {
           tma_load_3d(b_dst, &tmB, &full[stage], kb * GEMM_BK, n_blk * BN_OUT, expert);
@@ -207,6 +212,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 float f[8];
 #pragma unroll
                 for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(r[v * 8 + i]);
+                if (EPI == EPI_F32_DIAG) {
+                  float* dst = reinterpret_cast<float*>(C) + (size_t)row * ldc + col;
+                  *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
+                  *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
+                  continue;
+                }
                 if (EPI == EPI_ROWSCALE) {
 #pragma unroll
                   for (int i = 0; i < 8; ++i) f[i] *= row_scale;
@@ -267,7 +278,8 @@ struct GemmExtra {
   const int* tile_expert = nullptr;    // [max m tiles]
   const int* num_m_tiles = nullptr;    // device scalar
   int w_rows = 0;                      // rows of W per expert (N for plain epilogues, 2*n_half for EPI_SILU_SPLIT)
-  int n_half = 0;                      // EPI_SILU_SPLIT: row offset of the `up` half
+  int n_half = 0;                      // EPI_SILU_SPLIT: row offset of the `up` half; EPI_F32_DIAG: rows per block
+  int a_cols = 0;                      // EPI_F32_DIAG: columns of A (all blocks)
 };
 
 template <int BN, int EPI, bool GROUPED>
@@ -278,7 +290,7 @@ static void launch_gemm(const void* A, const void* W, void* C, const void* bias,
   constexpr int BN_OUT = SPLIT ? BN / 2 : BN;
   if (SPLIT && BN < 64) throw std::runtime_error("sglb gemm: split-silu epilogue needs BN >= 64");
   const int w_rows = ex.w_rows > 0 ? ex.w_rows : N;
-  uint64_t dA[2] = {(uint64_t)K, (uint64_t)M}, sAs[1] = {(uint64_t)lda * 2};
+  uint64_t dA[2] = {(uint64_t)(ex.a_cols > 0 ? ex.a_cols : K), (uint64_t)M}, sAs[1] = {(uint64_t)lda * 2};
   uint32_t bA[2] = {GEMM_BK, GEMM_BM};
   CUtensorMap tmA = make_tmap(A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dA, sAs, bA, CU_TENSOR_MAP_SWIZZLE_128B);
   CUtensorMap tmB;
@@ -361,6 +373,21 @@ void gemm_bf16_tc(const void* A, const void* W, void* C, const void* bias, int M
     }
     default: throw std::runtime_error("sglb gemm: bad epilogue");
   }
+}
+
+// block-diagonal product with an fp32 result: A [M, blocks * K], W [blocks * rows, K] -> C fp32 [M, blocks * rows]
+void gemm_bf16_tc_diag_f32(const void* A, const void* W, float* C, int M, int blocks, int rows, int K, int lda, int num_sms, cudaStream_t stream) {
+  if (M <= 0 || blocks <= 0) return;
+  if (K % 8 || rows % 32 || lda % 8) throw std::runtime_error("sglb block-diagonal gemm: K % 8, rows % 32, lda % 8 required");
+  GemmExtra ex; ex.n_half = rows; ex.a_cols = blocks * K;
+  const int N = blocks * rows, m_tiles = (M + GEMM_BM - 1) / GEMM_BM;
+  int bn = 32;
+  for (int cand : {128, 64, 32}) {
+    if (rows % cand) continue;
+    bn = cand;
+    if ((long long)m_tiles * (N / cand) >= num_sms) break;
+  }
+  dispatch_bn<EPI_F32_DIAG>(bn, A, W, C, nullptr, M, N, K, lda, K, N, num_sms, stream, GemmPush{}, ex);
 }
 
 // Expert-grouped GEMM over expert-sorted, 128-row-padded activations (see moe.cu for the alignment kernels).

@@ -29,11 +29,11 @@ template <> __device__ __forceinline__ void st_f<float>(float* p, float v) { *p 
 template <> __device__ __forceinline__ void st_f<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
 // grid (ceil(C / 256), chunks, B); thread = channel.  cu_q == nullptr: decode (one token per request, row = request index).
-template <typename T>
+template <typename T, typename TU>
 __global__ void __launch_bounds__(256) causal_conv1d_fwd_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, const T* __restrict__ bias,
                                                                 const T* __restrict__ conv_state, const int* __restrict__ cu_q,
                                                                 const int* __restrict__ req_slots, const int* __restrict__ seq_lens, int C, int K,
-                                                                int silu, float* __restrict__ u, int ldu) {
+                                                                int silu, TU* __restrict__ u, int ldu) {
   const int c = blockIdx.x * 256 + threadIdx.x;
   const int b = blockIdx.z;
   if (c >= C) return;
@@ -75,7 +75,7 @@ __global__ void __launch_bounds__(256) causal_conv1d_fwd_kernel(const T* __restr
       else if (j == K - 2) win[j] = xv;
     }
     if (silu) acc = acc / (1.f + __expf(-acc));
-    u[(size_t)(q0 + t) * ldu + c] = acc;
+    st_f<TU>(u + (size_t)(q0 + t) * ldu + c, acc);
   }
 }
 
@@ -138,17 +138,23 @@ void causal_conv1d_state(const void* x, int ldx, void* conv_state, const int* cu
 }
 
 void causal_conv1d(const void* x, int ldx, const void* w, const void* bias, void* conv_state, const int* cu_q, const int* req_slots,
-                   const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, float* u, int ldu, cudaStream_t stream) {
+                   const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, void* u, bool u_bf16, int ldu, cudaStream_t stream) {
   if (B <= 0) return;
   if (K < 2 || K > CONV_MAX_K) throw std::runtime_error("sglb causal_conv1d: kernel width must be 2..8");
+  if (u_bf16 && !bf16) throw std::runtime_error("sglb causal_conv1d: the output is fp32 or of the input's type");
   dim3 g1((C + 255) / 256, (std::max(max_q_len, 1) + CONV_CHUNK - 1) / CONV_CHUNK, B), g2((C + 255) / 256, B);
+  using bf = __nv_bfloat16;
   if (bf16) {
-    causal_conv1d_fwd_kernel<__nv_bfloat16><<<g1, 256, 0, stream>>>((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, (const __nv_bfloat16*)bias,
-                                                                    (const __nv_bfloat16*)conv_state, cu_q, req_slots, seq_lens, C, K, silu ? 1 : 0, u, ldu);
-    causal_conv1d_state_kernel<__nv_bfloat16><<<g2, 256, 0, stream>>>((const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)conv_state, cu_q, req_slots, seq_lens, C, K);
+    if (u_bf16)
+      causal_conv1d_fwd_kernel<bf, bf><<<g1, 256, 0, stream>>>((const bf*)x, ldx, (const bf*)w, (const bf*)bias, (const bf*)conv_state, cu_q, req_slots, seq_lens, C,
+                                                               K, silu ? 1 : 0, (bf*)u, ldu);
+    else
+      causal_conv1d_fwd_kernel<bf, float><<<g1, 256, 0, stream>>>((const bf*)x, ldx, (const bf*)w, (const bf*)bias, (const bf*)conv_state, cu_q, req_slots,
+                                                                  seq_lens, C, K, silu ? 1 : 0, (float*)u, ldu);
+    causal_conv1d_state_kernel<bf><<<g2, 256, 0, stream>>>((const bf*)x, ldx, (bf*)conv_state, cu_q, req_slots, seq_lens, C, K);
   } else {
-    causal_conv1d_fwd_kernel<float><<<g1, 256, 0, stream>>>((const float*)x, ldx, (const float*)w, (const float*)bias, (const float*)conv_state, cu_q,
-                                                            req_slots, seq_lens, C, K, silu ? 1 : 0, u, ldu);
+    causal_conv1d_fwd_kernel<float, float><<<g1, 256, 0, stream>>>((const float*)x, ldx, (const float*)w, (const float*)bias, (const float*)conv_state, cu_q,
+                                                                   req_slots, seq_lens, C, K, silu ? 1 : 0, (float*)u, ldu);
     causal_conv1d_state_kernel<float><<<g2, 256, 0, stream>>>((const float*)x, ldx, (float*)conv_state, cu_q, req_slots, seq_lens, C, K);
   }
   SGLB_CUDA_CHECK(cudaGetLastError());
@@ -516,6 +522,110 @@ void mamba2_scan(const float* u, int ldu, const void* z, int ldz, const void* dt
   p.req_slots = req_slots; p.seq_lens = seq_lens; p.cu_q = cu_q; p.out = out; p.H = H; p.P = P; p.N = N; p.G = G; p.pchunks = 1;
   if (bf16) dispatch_m2<__nv_bfloat16>(p, B, stream);
   else dispatch_m2<float>(p, B, stream);
+}
+
+// ---------------------------------------------------------------- inputs of a linear attention's scan
+// projection rows [v (H*Dv) | k (H*D) | q (H*D) | ...] -> fp32 rows [v | k | q]: optional SiLU, the first 2 * half coordinates of every k and q head
+// turned by position * inv_freq[m] (pairs (m, m + half), or neighbours), k times a constant.  One CTA per token; the token's sines and cosines
+// are computed once into shared memory and serve all heads.  VEC = 4: four columns per access.
+namespace {
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) linear_attention_prepare_kernel(const T* __restrict__ proj, int ld, int H, int D, int Dv, const int* __restrict__ positions,
+                                                                       const float* __restrict__ inv_freq, int half, int inter, float k_scale, int silu,
+                                                                       float* __restrict__ u) {
+  extern __shared__ float2 trig[];
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const T* row = proj + (size_t)t * ld;
+  const int nv = H * Dv, nk = H * D;
+  float* dst = u + (size_t)t * (nv + 2 * nk);
+  if (half > 0) {
+    const float pos = (float)positions[t];
+    for (int m = tid; m < half; m += 256) {
+      float sn, cs;
+      sincosf(pos * inv_freq[m], &sn, &cs);
+      trig[m] = make_float2(cs, sn);
+    }
+    __syncthreads();
+  }
+  struct V { float v[VEC]; };
+  auto load = [&](int c) {
+    V r;
+    if constexpr (VEC == 4) {
+      if constexpr (sizeof(T) == 2) {
+        const uint2 w = *reinterpret_cast<const uint2*>(row + c);
+        r.v[0] = bf16_lo(w.x); r.v[1] = bf16_hi(w.x); r.v[2] = bf16_lo(w.y); r.v[3] = bf16_hi(w.y);
+      } else {
+        const float4 w = *reinterpret_cast<const float4*>(row + c);
+        r.v[0] = w.x; r.v[1] = w.y; r.v[2] = w.z; r.v[3] = w.w;
+      }
+    } else r.v[0] = ld_f<T>(row + c);
+    if (silu) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) r.v[e] = r.v[e] / (1.f + expf(-r.v[e]));
+    }
+    return r;
+  };
+  auto store = [&](int c, const V& r) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst + c) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else dst[c] = r.v[0];
+  };
+  for (int c = tid * VEC; c < nv + 2 * nk; c += 256 * VEC) {
+    V r = load(c);
+    if (c >= nv) {
+      const int rel = c - nv;
+      const bool isk = rel < nk;
+      const int i = (isk ? rel : rel - nk) % D;
+      if (i < 2 * half) {
+        if (inter) {
+          if constexpr (VEC == 4) {
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+              const float2 cs = trig[(i + e) >> 1];
+              const float a = r.v[e], b = r.v[e + 1];
+              r.v[e] = a * cs.x - b * cs.y;
+              r.v[e + 1] = b * cs.x + a * cs.y;
+            }
+          } else {
+            const float2 cs = trig[i >> 1];
+            const float other = load(c + ((i & 1) ? -1 : 1)).v[0];
+            r.v[0] = (i & 1) ? r.v[0] * cs.x + other * cs.y : r.v[0] * cs.x - other * cs.y;
+          }
+        } else {
+          const bool first = i < half;
+          const V o = load(first ? c + half : c - half);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            const float2 cs = trig[(first ? i : i - half) + e];
+            r.v[e] = first ? r.v[e] * cs.x - o.v[e] * cs.y : r.v[e] * cs.x + o.v[e] * cs.y;
+          }
+        }
+      }
+      if (isk) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r.v[e] *= k_scale;
+      }
+    }
+    store(c, r);
+  }
+}
+
+}  // namespace
+
+void linear_attention_prepare(const void* proj, int ld, bool bf16, int T, int H, int D, int Dv, const int* positions, const float* inv_freq, int half,
+                              bool interleaved, float k_scale, bool silu, float* u, cudaStream_t stream) {
+  if (T <= 0) return;
+  const size_t smem = sizeof(float2) * (size_t)half;
+  if (smem > 48 * 1024) throw std::runtime_error("sglb linear_attention_prepare: rotary widths up to 12,288");
+  const bool vec = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && (2 * half) % 4 == 0 && (interleaved || half % 4 == 0) &&
+                   ((uintptr_t)proj % (bf16 ? 8 : 16)) == 0 && ((uintptr_t)u % 16) == 0;
+  const int in = interleaved ? 1 : 0, act = silu ? 1 : 0;
+#define SGLB_LAP(TT, V) \
+  linear_attention_prepare_kernel<TT, V><<<T, 256, smem, stream>>>((const TT*)proj, ld, H, D, Dv, positions, inv_freq, half, in, k_scale, act, u)
+  if (bf16) { if (vec) SGLB_LAP(__nv_bfloat16, 4); else SGLB_LAP(__nv_bfloat16, 1); }
+  else { if (vec) SGLB_LAP(float, 4); else SGLB_LAP(float, 1); }
+#undef SGLB_LAP
+  SGLB_CUDA_CHECK(cudaGetLastError());
 }
 
 // ---------------------------------------------------------------- matrix memory with exponential gates and a running maximum (mLSTM): what surrounds the scan

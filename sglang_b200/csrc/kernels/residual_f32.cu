@@ -3,6 +3,7 @@
 //   add_rmsnorm_f32 : residual (fp32, in place) += delta (bf16 | fp32 | none); out = residual / rms(residual) * (w | 1 + w) in bf16 | fp32.
 //                     One block per row; the sum, the mean of squares and the scaling are fp32, eps sits inside the root.  The weight is a
 //                     vector or one number for all coordinates.
+//   stream_mix_norm : several parallel fp32 streams instead of one (hyper-connections): mixing, the update and the next sublayer's normed input.
 //   clamped_glu     : [gate | up] halves -> min(g, limit) * sigmoid(alpha * g) * (clamp(u, -limit, limit) + 1), fp32 math.
 #include <stdexcept>
 
@@ -265,11 +266,17 @@ __global__ void __launch_bounds__(256) norm_add_f32_kernel(float* __restrict__ x
   }
 }
 
-// x fp32 [T, C] in ``groups`` equal parts: part / sqrt(mean(part^2) + eps) * w [* sigmoid(gate)] * out_scale; grid (T, groups); gate and out are
-// rows of ldg / ldo elements
+// gate activations of grouped_rmsnorm
+__device__ __forceinline__ float gate_act(float g, int silu) {
+  const float s = 1.f / (1.f + expf(-g));
+  return silu ? g * s : s;
+}
+
+// x fp32 [T, C] in ``groups`` equal parts: part / sqrt(mean(part^2) + eps) [* w] [* sigmoid(gate) | * silu(gate)] * out_scale; grid (T, groups); gate and
+// out are rows of ldg / ldo elements
 template <typename TO>
 __global__ void __launch_bounds__(256) grouped_rmsnorm_kernel(const float* __restrict__ x, const TO* __restrict__ w, TO* __restrict__ out, int C, int per,
-                                                              float eps, const TO* __restrict__ gate, int ldg, int ldo, float out_scale) {
+                                                              float eps, const TO* __restrict__ gate, int ldg, int ldo, float out_scale, int silu) {
   __shared__ float red[8];
   const size_t base = (size_t)blockIdx.x * C + (size_t)blockIdx.y * per;
   float ss = 0.f;
@@ -282,36 +289,243 @@ __global__ void __launch_bounds__(256) grouped_rmsnorm_kernel(const float* __res
   TO* o = out + (size_t)blockIdx.x * ldo + c0;
   const TO* gr = gate ? gate + (size_t)blockIdx.x * ldg + c0 : nullptr;
   for (int i = threadIdx.x; i < per; i += 256) {
-    float v = x[base + i] * rs * ldf<TO>(w + c0 + i);
-    if (gr) v *= 1.f / (1.f + expf(-ldf<TO>(gr + i)));
+    float v = x[base + i] * rs;
+    if (w) v *= ldf<TO>(w + c0 + i);
+    if (gr) v *= gate_act(ldf<TO>(gr + i), silu);
     stf<TO>(o + i, v);
   }
 }
 
-// the same with one warp per (row, part): a CTA of 8 warps walks the parts of its row (many small parts: no CTA-wide barrier, 16-byte loads)
+// the same with one warp per (row, part): a CTA of 8 warps walks the parts of its row (many small parts: no CTA-wide barrier, four columns per
+// access); a part of up to 512 columns stays in registers between the two passes
 template <typename TO>
 __global__ void __launch_bounds__(256) grouped_rmsnorm_warp_kernel(const float* __restrict__ x, const TO* __restrict__ w, TO* __restrict__ out, int C,
-                                                                   int per, int groups, float eps) {
+                                                                   int per, int groups, float eps, const TO* __restrict__ gate, int ldg, int ldo,
+                                                                   float out_scale, int silu) {
+  constexpr int KEEP = 4;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n4 = per / 4;
   for (int g = warp; g < groups; g += 8) {
-    const size_t base = (size_t)blockIdx.x * C + (size_t)g * per;
-    const float4* xv = reinterpret_cast<const float4*>(x + base);
+    const float4* xv = reinterpret_cast<const float4*>(x + (size_t)blockIdx.x * C + (size_t)g * per);
+    float4 keep[KEEP];
     float ss = 0.f;
-    for (int i = lane; i < per / 4; i += 32) {
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = lane + k * 32;
+      keep[k] = i < n4 ? xv[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += keep[k].x * keep[k].x + keep[k].y * keep[k].y + keep[k].z * keep[k].z + keep[k].w * keep[k].w;
+    }
+    for (int i = lane + KEEP * 32; i < n4; i += 32) {
       const float4 v = xv[i];
       ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
-    const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)per + eps);
-    const TO* wr = w + (size_t)g * per;
-    for (int i = lane; i < per / 4; i += 32) {
-      const float4 v = xv[i];
-      TO* o = out + base + 4 * i;
-      stf<TO>(o, v.x * rs * ldf<TO>(wr + 4 * i));
-      stf<TO>(o + 1, v.y * rs * ldf<TO>(wr + 4 * i + 1));
-      stf<TO>(o + 2, v.z * rs * ldf<TO>(wr + 4 * i + 2));
-      stf<TO>(o + 3, v.w * rs * ldf<TO>(wr + 4 * i + 3));
+    const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)per + eps) * out_scale;
+    const size_t c0 = (size_t)g * per;
+    auto emit = [&](int i, float4 v) {
+      v.x *= rs; v.y *= rs; v.z *= rs; v.w *= rs;
+      if (w) {
+        const float4 a = ld4f<TO>(w + c0 + 4 * i);
+        v.x *= a.x; v.y *= a.y; v.z *= a.z; v.w *= a.w;
+      }
+      if (gate) {
+        const float4 a = ld4f<TO>(gate + (size_t)blockIdx.x * ldg + c0 + 4 * i);
+        v.x *= gate_act(a.x, silu); v.y *= gate_act(a.y, silu); v.z *= gate_act(a.z, silu); v.w *= gate_act(a.w, silu);
+      }
+      st4f<TO>(out + (size_t)blockIdx.x * ldo + c0 + 4 * i, v);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = lane + k * 32;
+      if (i < n4) emit(i, keep[k]);
+    }
+    for (int i = lane + KEEP * 32; i < n4; i += 32) emit(i, xv[i]);
+  }
+}
+
+// S parallel fp32 residual streams x [T, S, W] (hyper-connections).  coef = mix [from, to] (S x S) | out (S) | in (S):
+//   x'_t = sum_s mix[s, t] x_s + out[t] y      all streams from the old ones (without y: x' = x);   written to xn when given
+//   u    = sum_t in[t] x'_t;   h = (u - mean) / sqrt(mean((u - mean)^2) + eps) * w       (centre = 0: u / sqrt(mean(u^2) + eps) * w)
+// x == nullptr: every old stream is the embedding row table[ids].  One CTA per token; a thread owns the same columns of every stream, so x' may
+// replace x in place.  u stays in registers (4 accesses per thread) and, for wider rows, in shared memory; mean and variance are two passes.
+// SN: number of streams at compile time (0: at run time, up to 16).  VEC = 4: four columns per access.
+template <int VEC> struct StreamVec;
+template <> struct StreamVec<1> {
+  float v[1];
+};
+template <> struct StreamVec<4> {
+  float v[4];
+};
+template <int VEC> __device__ __forceinline__ StreamVec<VEC> sv_ld(const float* p) {
+  StreamVec<VEC> r;
+  if constexpr (VEC == 4) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w;
+  } else r.v[0] = *p;
+  return r;
+}
+template <int VEC> __device__ __forceinline__ StreamVec<VEC> sv_ld(const __nv_bfloat16* p) {
+  StreamVec<VEC> r;
+  if constexpr (VEC == 4) {
+    const float4 t = ld4f<__nv_bfloat16>(p);
+    r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w;
+  } else r.v[0] = __bfloat162float(*p);
+  return r;
+}
+template <int VEC> __device__ __forceinline__ void sv_st(float* p, const StreamVec<VEC>& r) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  else *p = r.v[0];
+}
+template <int VEC> __device__ __forceinline__ void sv_st(__nv_bfloat16* p, const StreamVec<VEC>& r) {
+  if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r.v[0], r.v[1]), pack_bf16(r.v[2], r.v[3]));
+  else *p = __float2bfloat16(r.v[0]);
+}
+
+constexpr int STREAM_MAX = 16;
+template <int SN> constexpr int STREAM_KEEP = SN > 0 ? 4 : 0;          // accesses per thread whose u stays in registers
+
+template <typename T, int SN, int VEC>
+__global__ void __launch_bounds__(256) stream_mix_norm_kernel(const float* x, const T* __restrict__ table, const int* __restrict__ ids, int rows,
+                                                              const T* __restrict__ y, const float* __restrict__ coef, int streams, const T* __restrict__ w,
+                                                              float* xn, T* __restrict__ h, int W, float eps, int centre) {
+  constexpr int SM = SN > 0 ? SN : STREAM_MAX;
+  constexpr int KEEP = STREAM_KEEP<SN>;
+  const int S = SN > 0 ? SN : streams;
+  extern __shared__ float su[];                     // u beyond the registers' columns
+  __shared__ float red[8];
+  __shared__ float sc[SM * SM + 2 * SM];
+  for (int i = threadIdx.x; i < S * S + 2 * S; i += 256) sc[i] = coef[i];
+  __syncthreads();
+  const float* cout = sc + S * S;
+  const float* cin = cout + S;
+  const int t = blockIdx.x;
+  const float* xr = x ? x + (size_t)t * S * W : nullptr;
+  const T* er = x ? nullptr : table + (size_t)min(max(ids[t], 0), rows - 1) * W;
+  const T* yr = y ? y + (size_t)t * W : nullptr;
+  float* nr = xn ? xn + (size_t)t * S * W : nullptr;
+
+  auto form = [&](int i) {                          // columns i .. i + VEC - 1: the new streams, and their weighted sum
+    StreamVec<VEC> u, yv, old[SM];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) u.v[e] = 0.f;
+    if (yr) yv = sv_ld<VEC>(yr + i);
+    if (xr) {
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) old[s] = sv_ld<VEC>(xr + (size_t)s * W + i);
+    } else {
+      const StreamVec<VEC> e = sv_ld<VEC>(er + i);
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) old[s] = e;
+    }
+#pragma unroll(SN > 0 ? SM : 1)
+    for (int d = 0; d < S; ++d) {
+      StreamVec<VEC> nv;
+      if (yr) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) nv.v[e] = cout[d] * yv.v[e];
+#pragma unroll
+        for (int s = 0; s < SM; ++s) {
+          if (s < S) {
+            const float m = sc[s * S + d];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) nv.v[e] += m * old[s].v[e];
+          }
+        }
+      } else if constexpr (SN > 0) nv = old[d];
+      else nv = xr ? sv_ld<VEC>(xr + (size_t)d * W + i) : old[0];
+      if (nr) sv_st<VEC>(nr + (size_t)d * W + i, nv);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) u.v[e] += cin[d] * nv.v[e];
+    }
+    return u;
+  };
+
+  StreamVec<VEC> keep[KEEP > 0 ? KEEP : 1];
+  constexpr int KCOLS = KEEP * 256 * VEC;
+  float sum = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (threadIdx.x + k * 256) * VEC;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) keep[k].v[e] = 0.f;
+    if (i < W) {
+      keep[k] = form(i);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sum += keep[k].v[e];
     }
   }
+  for (int i = KCOLS + threadIdx.x * VEC; i < W; i += 256 * VEC) {
+    const StreamVec<VEC> u = form(i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) { su[i - KCOLS + e] = u.v[e]; sum += u.v[e]; }
+  }
+  const float mean = centre ? block_sum_256(sum, red) / (float)W : 0.f;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (threadIdx.x + k * 256) * VEC;
+    if (i < W) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) { keep[k].v[e] -= mean; ss += keep[k].v[e] * keep[k].v[e]; }
+    }
+  }
+  for (int i = KCOLS + threadIdx.x * VEC; i < W; i += 256 * VEC) {          // each thread re-reads what it wrote
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) { const float d = su[i - KCOLS + e] - mean; ss += d * d; }
+  }
+  const float rs = 1.0f / sqrtf(block_sum_256(ss, red) / (float)W + eps);
+  T* hr = h + (size_t)t * W;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (threadIdx.x + k * 256) * VEC;
+    if (i < W) {
+      const StreamVec<VEC> a = sv_ld<VEC>(w + i);
+      StreamVec<VEC> o;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) o.v[e] = keep[k].v[e] * rs * a.v[e];
+      sv_st<VEC>(hr + i, o);
+    }
+  }
+  for (int i = KCOLS + threadIdx.x * VEC; i < W; i += 256 * VEC) {
+    const StreamVec<VEC> a = sv_ld<VEC>(w + i);
+    StreamVec<VEC> o;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) o.v[e] = (su[i - KCOLS + e] - mean) * rs * a.v[e];
+    sv_st<VEC>(hr + i, o);
+  }
+}
+
+template <typename T, int SN, int VEC>
+void launch_stream_mix(const float* x, const T* table, const int* ids, int rows, const T* y, const float* coef, int S, const T* w, float* xn, T* h, int n,
+                       int W, float eps, bool centre, cudaStream_t stream) {
+  const int over = W - STREAM_KEEP<SN> * 256 * VEC;
+  const size_t smem = over > 0 ? sizeof(float) * (size_t)over : 0;
+  if (smem > 200 * 1024) throw std::runtime_error("sglb stream_mix_norm: rows up to 52,000 columns");
+  auto kern = stream_mix_norm_kernel<T, SN, VEC>;
+  if (smem > 32 * 1024) SGLB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<n, 256, smem, stream>>>(x, table, ids, rows, y, coef, S, w, xn, h, W, eps, centre ? 1 : 0);
+  SGLB_CUDA_CHECK(cudaGetLastError());
+}
+
+template <typename T>
+void dispatch_stream_mix(const float* x, const T* table, const int* ids, int rows, const T* y, const float* coef, int S, const T* w, float* xn, T* h, int n,
+                         int W, float eps, bool centre, cudaStream_t stream) {
+  auto al = [](const void* p) { return p == nullptr || ((uintptr_t)p % 16) == 0; };
+  const bool vec = W % 4 == 0 && al(x) && al(table) && al(y) && al(w) && al(xn) && al(h);
+#define SGLB_SM(SN)                                                                                                                       \
+  do {                                                                                                                                    \
+    if (vec) launch_stream_mix<T, SN, 4>(x, table, ids, rows, y, coef, S, w, xn, h, n, W, eps, centre, stream);                             \
+    else launch_stream_mix<T, SN, 1>(x, table, ids, rows, y, coef, S, w, xn, h, n, W, eps, centre, stream);                                 \
+  } while (0)
+  switch (S) {
+    case 1: SGLB_SM(1); break;
+    case 2: SGLB_SM(2); break;
+    case 3: SGLB_SM(3); break;
+    case 4: SGLB_SM(4); break;
+    default: SGLB_SM(0);
+  }
+#undef SGLB_SM
 }
 
 }  // namespace
@@ -376,22 +590,32 @@ void parallel_add_rmsnorm_f32(float* residual, const void* d1, const void* d2, b
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
 
+void stream_mix_norm(const float* x, const void* table, const int* ids, int rows, const void* y, const float* coef, int streams, const void* w, float* xn,
+                     void* h, bool bf16, int T, int W, float eps, bool centre, cudaStream_t stream) {
+  if (T <= 0 || W <= 0) return;
+  if (streams < 1 || streams > STREAM_MAX) throw std::runtime_error("sglb stream_mix_norm: 1 to 16 streams");
+  using bf = __nv_bfloat16;
+  if (bf16) dispatch_stream_mix<bf>(x, (const bf*)table, ids, rows, (const bf*)y, coef, streams, (const bf*)w, xn, (bf*)h, T, W, eps, centre, stream);
+  else dispatch_stream_mix<float>(x, (const float*)table, ids, rows, (const float*)y, coef, streams, (const float*)w, xn, (float*)h, T, W, eps, centre, stream);
+}
+
 void grouped_rmsnorm(const float* x, const void* w, void* out, bool out_bf16, int T, int C, int groups, float eps, const void* gate, int ldg, int ldo,
-                     float out_scale, cudaStream_t stream) {
+                     float out_scale, bool silu, cudaStream_t stream) {
   if (T <= 0) return;
   if (groups <= 0 || C % groups || groups > 65535) throw std::runtime_error("sglb grouped_rmsnorm: the width must split into equal parts");
-  const int per = C / groups;
-  if (!gate && ldo == C && out_scale == 1.f && groups >= 4 && per % 4 == 0 && per <= 4096 && ((uintptr_t)x % 16) == 0) {
-    if (out_bf16) grouped_rmsnorm_warp_kernel<__nv_bfloat16><<<T, 256, 0, stream>>>(x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, C, per, groups, eps);
-    else grouped_rmsnorm_warp_kernel<float><<<T, 256, 0, stream>>>(x, (const float*)w, (float*)out, C, per, groups, eps);
+  const int per = C / groups, act = silu ? 1 : 0;
+  const size_t a4 = out_bf16 ? 8 : 16;               // bytes of a four-column access
+  auto al = [&](const void* p) { return p == nullptr || ((uintptr_t)p % a4) == 0; };
+  using bf = __nv_bfloat16;
+  if (groups >= 4 && per % 4 == 0 && per <= 4096 && ldo % 4 == 0 && (!gate || ldg % 4 == 0) && ((uintptr_t)x % 16) == 0 && al(w) && al(out) && al(gate)) {
+    if (out_bf16) grouped_rmsnorm_warp_kernel<bf><<<T, 256, 0, stream>>>(x, (const bf*)w, (bf*)out, C, per, groups, eps, (const bf*)gate, ldg, ldo, out_scale, act);
+    else grouped_rmsnorm_warp_kernel<float><<<T, 256, 0, stream>>>(x, (const float*)w, (float*)out, C, per, groups, eps, (const float*)gate, ldg, ldo, out_scale, act);
     SGLB_CUDA_CHECK(cudaGetLastError());
     return;
   }
   dim3 g(T, groups);
-  if (out_bf16)
-    grouped_rmsnorm_kernel<__nv_bfloat16><<<g, 256, 0, stream>>>(x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, C, per, eps, (const __nv_bfloat16*)gate, ldg,
-                                                                 ldo, out_scale);
-  else grouped_rmsnorm_kernel<float><<<g, 256, 0, stream>>>(x, (const float*)w, (float*)out, C, per, eps, (const float*)gate, ldg, ldo, out_scale);
+  if (out_bf16) grouped_rmsnorm_kernel<bf><<<g, 256, 0, stream>>>(x, (const bf*)w, (bf*)out, C, per, eps, (const bf*)gate, ldg, ldo, out_scale, act);
+  else grouped_rmsnorm_kernel<float><<<g, 256, 0, stream>>>(x, (const float*)w, (float*)out, C, per, eps, (const float*)gate, ldg, ldo, out_scale, act);
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
 

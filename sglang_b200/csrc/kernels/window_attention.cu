@@ -458,7 +458,7 @@ struct PrepParams {
   int H, G, D, Dv;
   const int* positions;
   const void* qw; const void* kw; float eps;   // projection-wide RMS norm weights (null: no norm)
-  const float* inv_freq; int half;             // rotary frequencies (null: no rotation); pairs (i, i + half), i < half
+  const float* inv_freq; int half; int inter;  // rotary frequencies (null: no rotation); pairs (i, i + half), i < half, or, inter, (2i, 2i + 1)
   const void* v_first; int ldvf; float lam;    // values to blend with (null: none)
   const float* v_inv_freq; int v_inter;        // values rotated over their whole head (null: no): pairs (m, m + Dv/2) or, v_inter, (2m, 2m + 1)
   void* kc; void* vc; size_t ldc; const int* loc;
@@ -506,11 +506,12 @@ __global__ void __launch_bounds__(128) attention_prepare_kernel(const PrepParams
     auto val = [&](int c) { const float v = wa_ld<T>(src + c) * r; return w ? v * wa_ld<T>(w + hd * p.D + c) : v; };
     float v = val(i);
     if (i < 2 * half) {
-      const int fi = i < half ? i : i - half;
+      const bool first = p.inter ? (i & 1) == 0 : i < half;
+      const int fi = p.inter ? i >> 1 : first ? i : i - half;
       float sn, cs;
       sincosf(pos * p.inv_freq[fi], &sn, &cs);
-      const float other = val(i < half ? i + half : i - half);
-      v = i < half ? v * cs - other * sn : v * cs + other * sn;
+      const float other = val(p.inter ? i ^ 1 : first ? i + half : i - half);
+      v = first ? v * cs - other * sn : v * cs + other * sn;
     }
     wa_st<T>(dst, v);
   }
@@ -549,7 +550,8 @@ __device__ __forceinline__ void wa_st2(float* p, float a, float b) { *reinterpre
 __device__ __forceinline__ void wa_st2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b); }
 
 // the same work two columns at a time: even head sizes, rotary half-width and strides.  A rotated item is the four numbers
-// (i, i + 1, i + half, i + half + 1) of a head: two angles, each pair rotated once; a tail item is two unrotated columns (or zero padding).
+// (i, i + 1, i + half, i + half + 1) of a head: two angles, each pair rotated once (neighbouring pairs: the two numbers of one pair); a tail item is
+// two unrotated columns (or zero padding).
 template <typename T>
 __global__ void __launch_bounds__(128) attention_prepare_vec_kernel(const PrepParams p) {
   __shared__ float red[8];
@@ -576,7 +578,7 @@ __global__ void __launch_bounds__(128) attention_prepare_vec_kernel(const PrepPa
   T* ko = reinterpret_cast<T*>(p.kc) + slot * p.ldc;
   T* vo = reinterpret_cast<T*>(p.vc) + slot * p.ldc;
   const int half = p.inv_freq ? p.half : 0;
-  const int nrot = half / 2;                              // rotated items per head
+  const int nrot = p.inter ? half : half / 2;             // rotated items per head
   const int per_q = nrot + (p.Dq - 2 * half) / 2, per_k = nrot + (p.hsk - 2 * half) / 2;
   const int total = p.H * per_q + p.G * per_k;
   for (int idx = tid; idx < total; idx += 128) {
@@ -594,7 +596,12 @@ __global__ void __launch_bounds__(128) attention_prepare_vec_kernel(const PrepPa
       if (w) { const float2 ww = wa_ld2(w + hd * p.D + c); v.x *= ww.x; v.y *= ww.y; }
       return v;
     };
-    if (it < nrot) {
+    if (it < nrot && p.inter) {
+      const float2 a = val2(2 * it);
+      float sn, cs;
+      sincosf(pos * p.inv_freq[it], &sn, &cs);
+      wa_st2(dst + 2 * it, a.x * cs - a.y * sn, a.y * cs + a.x * sn);
+    } else if (it < nrot) {
       const int i = 2 * it;
       const float2 a = val2(i), b = val2(i + half);
       float s0, c0, s1, c1;
@@ -659,16 +666,17 @@ void sigmoid_gate(const void* o, int head_stride, const void* gate, int ldg, boo
 
 void attention_prepare(const void* qkv, int ld, bool bf16, int T, int H, int G, int D, int Dv, const int* positions, const void* q_norm_w, const void* k_norm_w,
                        float eps, const float* inv_freq, int half, const void* v_first, int ldvf, float lam, void* kc, void* vc, size_t ldc, const int* loc,
-                       void* q_out, int pad, const float* v_inv_freq, bool v_interleaved, cudaStream_t stream) {
+                       void* q_out, int pad, const float* v_inv_freq, bool v_interleaved, bool interleaved, cudaStream_t stream) {
   if (T <= 0) return;
   PrepParams p;
+  p.inter = interleaved ? 1 : 0;
   p.v_inv_freq = v_inv_freq; p.v_inter = v_interleaved ? 1 : 0;
   p.qkv = qkv; p.ld = ld; p.H = H; p.G = G; p.D = D; p.Dv = Dv; p.positions = positions; p.qw = q_norm_w; p.kw = k_norm_w; p.eps = eps;
   p.inv_freq = inv_freq; p.half = half; p.v_first = v_first; p.ldvf = ldvf; p.lam = lam; p.kc = kc; p.vc = vc; p.ldc = ldc; p.loc = loc; p.q_out = q_out;
   p.Dq = pad > 0 ? pad : D; p.hsk = pad > 0 ? pad : D; p.hsv = pad > 0 ? pad : Dv;
   const size_t a2 = bf16 ? 4 : 8;          // bytes of a two-element access
   auto al = [&](const void* q) { return q == nullptr || ((uintptr_t)q % a2) == 0; };
-  const bool vec = D % 2 == 0 && Dv % 2 == 0 && half % 2 == 0 && ld % 2 == 0 && ldc % 2 == 0 && p.Dq % 2 == 0 && p.hsk % 2 == 0 && p.hsv % 2 == 0 &&
+  const bool vec = D % 2 == 0 && Dv % 2 == 0 && (interleaved || half % 2 == 0) && ld % 2 == 0 && ldc % 2 == 0 && p.Dq % 2 == 0 && p.hsk % 2 == 0 && p.hsv % 2 == 0 &&
                    (v_inv_freq == nullptr || v_interleaved || Dv % 4 == 0) && (v_first == nullptr || ldvf % 2 == 0) && al(qkv) && al(kc) && al(vc) && al(q_out) && al(v_first) && al(q_norm_w) && al(k_norm_w);
   if (vec) {
     if (bf16) attention_prepare_vec_kernel<__nv_bfloat16><<<T, 128, 0, stream>>>(p);

@@ -1,9 +1,9 @@
 """Grouped-query attention with an output gate, whose other parts are switched on by its arguments:
 
-    q, k, v, g = W h (+ b)                        one GEMM, rows [q | k | v | g]
+    q, k, v, g = W h (+ b)                        one GEMM, rows [q | k | v | g]; ``bias`` also gives the output projection one unless ``out_bias`` is False
     q, k       <- rms(q) * w_q, rms(k) * w_k      ``qk_norm``: over the WHOLE projection (all heads at once), plain weights
     q, k       <- rotation by position            ``rotary = (dims, inv_freq)``: the first ``dims`` coordinates of every head, coordinate i paired
-                                                  with i + dims/2, angle = position * inv_freq[i] (fp32)
+                                                  with i + dims/2 (``interleaved``: 2i with 2i + 1), angle = position * inv_freq[i] (fp32)
     v          <- (1 - lam) v + lam v_first       ``value_mix``: v_first = the values of the first such layer for the same token; the blend is cached
     v_j        <- v_j turned by position j        ``value_rotary = (inv_freq, interleaved)``: over the whole head, cached so; o_i is turned back by
                                                   position i behind the soft-max, so that a value enters by its distance to the query
@@ -66,7 +66,7 @@ class GatedAttention(nn.Module):
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: Optional[float], eps: float, dtype, *, bias: bool = False,
                  qk_norm: bool = False, rotary: Optional[Tuple[int, torch.Tensor]] = None, window: int = -1, keep_first: int = 0,
                  log_bias: bool = False, gate: Optional[str] = "head", value_mix: bool = False, own_projection: bool = True, softcap: float = 0.0,
-                 sinks: bool = False, value_rotary: Optional[Tuple[torch.Tensor, bool]] = None):
+                 sinks: bool = False, value_rotary: Optional[Tuple[torch.Tensor, bool]] = None, interleaved: bool = False, out_bias: Optional[bool] = None):
         super().__init__()
         assert heads % kv_heads == 0 and gate in ("head", "element", None)
         self.H, self.G, self.D, self.Dv, self.eps = heads, kv_heads, dim, vdim, eps
@@ -89,11 +89,11 @@ class GatedAttention(nn.Module):
         self.in_weight = mk(self.rows, width) if own_projection else None
         self.in_bias = mk(self.rows) if own_projection and bias else None
         self.o_weight = mk(width, heads * vdim)
-        self.o_bias = mk(width) if bias else None
+        self.o_bias = mk(width) if (bias if out_bias is None else out_bias) else None
         self.q_norm = mk(self.n_q) if qk_norm else None
         self.k_norm = mk(self.n_k) if qk_norm else None
         self.r1, self.r2 = (f32(heads), f32(heads)) if log_bias else (None, None)
-        self.rot_dims = int(rotary[0]) if rotary else 0
+        self.rot_dims, self.interleaved = int(rotary[0]) if rotary else 0, bool(interleaved)
         assert self.rot_dims % 2 == 0 and self.rot_dims <= dim
         self.inv_freq = nn.Parameter(rotary[1].float().clone(), requires_grad=False) if rotary else None
         self.vmix = 0.0              # lam (read when this layer is not the first value-mixing one)
@@ -160,7 +160,7 @@ class GatedAttention(nn.Module):
         kc, vc = planes if planes is not None else (fb.kv_pool.k(cache_idx), fb.kv_pool.v(cache_idx))      # [slots, 1, cache_width] each
         pad = self.pad
         q = ops.attention_prepare(proj, H, G, D, Dv, fb.positions, kc, vc, fb.out_cache_loc, self.q_norm, self.k_norm, self.eps, self.inv_freq,
-                                  v_first if self.value_mix else None, self.vmix, pad, self.v_inv_freq, self.v_interleaved)
+                                  v_first if self.value_mix else None, self.vmix, pad, self.v_inv_freq, self.v_interleaved, self.interleaved)
         gate = proj[:, self.rows - self.n_g:self.rows] if self.n_g else None
         turn = self.v_inv_freq is not None
         # where the back-rotation may write the caller's buffer directly: nothing follows it

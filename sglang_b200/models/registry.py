@@ -157,6 +157,9 @@ def _register_builtins() -> None:
     from . import mumasun as _mm
 
     register_model("Mumasun", _mm.MumasunForCausalLM)
+    from . import surasun as _su
+
+    register_model("Surasun", _su.SurasunForCausalLM)
     from . import transformers_fallback as _tff
 
     register_model("TransformersForCausalLM", _tff.TransformersForCausalLM)

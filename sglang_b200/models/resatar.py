@@ -41,6 +41,7 @@ from ..layers.gated_attention import GatedAttention, scaled_inv_freq
 from ..layers.linear_attention import DecayLinearAttention
 from ..layers.mamba1_scan import Mamba1ScanMixer
 from ..layers.moe import FusedMoE, select_experts
+from ..layers.parallel_mixer import ParallelMixer
 from ..layers.window_attention import FlatCacheSpec
 from ..mem_cache.memory_pool import LayeredStatePool
 from ..model_executor.forward_batch import ForwardBatch
@@ -118,51 +119,15 @@ class BiasedTopKMoE(nn.Module):
         return moe_ops.moe_identity_shared_combine(y.contiguous(), h, None, self.shared(h), None)
 
 
-class ParallelMixer(nn.Module):
-    """``left_scale * window attention + right_scale * decaying linear attention`` on the same input: one projection GEMM with rows
-    [left q | k | v | g | right v | k | q | g], and one output GEMM over the two sides' gated heads side by side (the constants folded into
-    the epilogues that produce them, the left output bias times its constant added by the GEMM)"""
-
-    def __init__(self, width: int, m: dict, eps: float, dtype):
-        super().__init__()
-        a, b = m["left"], m["right"]
-        mask = a.get("mask") or {}
-        self.left = GatedAttention(width, int(a["heads"]), int(a.get("kv_heads", a["heads"])), int(a["dim"]), int(a.get("vdim", a["dim"])), a.get("scale"),
-                                   eps, dtype, bias=True, qk_norm=True, window=int(mask.get("size") or -1), keep_first=int(mask.get("keep_first") or 0),
-                                   log_bias=True, gate="element", own_projection=False)
-        self.right = DecayLinearAttention(width, int(b["heads"]), int(b["dim"]), int(b.get("vdim", b["dim"])), b["decay"], eps, dtype, own_projection=False)
-        self.left.out_scale, self.right.out_scale = float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0))
-        self.left.o_weight = self.left.o_bias = self.right.o_weight = None          # they live in ``o_weight`` / ``o_bias`` below
-        nl, nr = self.left.rows, self.right.rows
-        self.in_weight = nn.Parameter(torch.zeros(nl + nr, width, dtype=dtype), requires_grad=False)
-        self.in_bias = nn.Parameter(torch.zeros(nl + nr, dtype=dtype), requires_grad=False)
-        self.n_ol, self.n_or = self.left.H * self.left.Dv, self.right.n_v
-        self.o_weight = nn.Parameter(torch.zeros(width, self.n_ol + self.n_or, dtype=dtype), requires_grad=False)
-        self.o_bias = nn.Parameter(torch.zeros(width, dtype=dtype), requires_grad=False)       # left output bias times left_scale
-
-    def load(self, leaf: str, w: torch.Tensor) -> bool:
-        side, _, rest = leaf.partition(".")
-        if side == "left":
-            if rest == "o":
-                self.o_weight.data[:, :self.n_ol].copy_(w)
-                return True
-            if rest == "o.b":
-                self.o_bias.data.copy_((w.float() * self.left.out_scale).to(self.o_bias.dtype))
-                return True
-            return self.left.load_in(rest, w, self.in_weight, self.in_bias, 0) or self.left.load(rest, w)
-        if side == "right":
-            if rest == "o":
-                self.o_weight.data[:, self.n_ol:].copy_(w)
-                return True
-            return self.right.load_in(rest, w, self.in_weight, None, self.left.rows) or self.right.load(rest, w)
-        return False
-
-    def forward(self, h: torch.Tensor, fb: ForwardBatch, cache_idx: int, state_idx: int) -> torch.Tensor:
-        proj = ops.linear(h, self.in_weight, self.in_bias)
-        cat = torch.empty(h.shape[0], self.n_ol + self.n_or, dtype=h.dtype, device=h.device)
-        self.left.attend(proj[:, :self.left.rows], fb, cache_idx, None, cat[:, :self.n_ol])
-        self.right.attend(proj[:, self.left.rows:], fb, state_idx, cat[:, self.n_ol:])
-        return ops.linear(cat, self.o_weight, self.o_bias)
+def parallel_mixer(width: int, m: dict, eps: float, dtype) -> ParallelMixer:
+    """``left_scale * window attention + right_scale * decaying linear attention`` on the same input"""
+    a, b = m["left"], m["right"]
+    mask = a.get("mask") or {}
+    left = GatedAttention(width, int(a["heads"]), int(a.get("kv_heads", a["heads"])), int(a["dim"]), int(a.get("vdim", a["dim"])), a.get("scale"),
+                          eps, dtype, bias=True, qk_norm=True, window=int(mask.get("size") or -1), keep_first=int(mask.get("keep_first") or 0),
+                          log_bias=True, gate="element", own_projection=False)
+    right = DecayLinearAttention(width, int(b["heads"]), int(b["dim"]), int(b.get("vdim", b["dim"])), b["decay"], eps, dtype, own_projection=False)
+    return ParallelMixer(width, left, right, float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0)), dtype)
 
 
 class ResatarBlock(nn.Module):
@@ -178,7 +143,7 @@ class ResatarBlock(nn.Module):
             self.mix = GatedAttention(W, int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m.get("vdim", m["dim"])), m.get("scale"),
                                       eps, dtype, rotary=rotary, gate="head", value_mix=bool(m.get("v_mix")))
         elif kind == "parallel":
-            self.mix = ParallelMixer(W, m, eps, dtype)
+            self.mix = parallel_mixer(W, m, eps, dtype)
         elif kind == "mamba1":
             self.mix = Mamba1ScanMixer(W, int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m.get("conv", 1)), dtype)
         else:

@@ -364,13 +364,14 @@ def sample(logits, temperature, top_k, top_p, min_p, seeds=None, out_slots=None,
 
 
 def causal_conv1d(x: torch.Tensor, w: torch.Tensor, bias, conv_state: torch.Tensor, cu_q, req_slots: torch.Tensor, seq_lens: torch.Tensor,
-                  max_q_len: int = 1, silu: bool = True) -> torch.Tensor:
-    """Mamba causal depthwise conv1d over a ragged batch, rolling state updated in place (csrc/kernels/mamba.cu); fp32 [T, C] out"""
-    if _use_native(x) and x.dtype in (torch.bfloat16, torch.float32) and x.stride(1) == 1 and 2 <= w.shape[1] <= 8:
-        u = torch.empty(x.shape[0], x.shape[1], dtype=torch.float32, device=x.device)
+                  max_q_len: int = 1, silu: bool = True, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """Mamba causal depthwise conv1d over a ragged batch, rolling state updated in place (csrc/kernels/mamba.cu); [T, C] out in fp32, or in the
+    input's dtype (``out_dtype``)"""
+    if _use_native(x) and x.dtype in (torch.bfloat16, torch.float32) and x.stride(1) == 1 and 2 <= w.shape[1] <= 8 and out_dtype in (torch.float32, x.dtype):
+        u = torch.empty(x.shape[0], x.shape[1], dtype=out_dtype, device=x.device)
         torch.ops.sglb.causal_conv1d(x, w.contiguous(), bias, conv_state, cu_q, req_slots, seq_lens, int(max_q_len), bool(silu), u)
         return u
-    return torch_ref.causal_conv1d(x, w, bias, conv_state, cu_q, req_slots, seq_lens, silu)
+    return torch_ref.causal_conv1d(x, w, bias, conv_state, cu_q, req_slots, seq_lens, silu).to(out_dtype)
 
 
 def selective_state_update(state: torch.Tensor, req_slots: torch.Tensor, x: torch.Tensor, dt: torch.Tensor, A: torch.Tensor, Bm: torch.Tensor,
@@ -556,19 +557,20 @@ def bigram_embedding(embed: torch.Tensor, bigram: Optional[torch.Tensor], ids: t
     return torch_ref.bigram_embedding(embed, bigram, ids, prev_tokens, cu_q, req_slots, seq_lens, scale, mul_prev, mul_cur, buckets)
 
 
-def grouped_rmsnorm(x: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, out_dtype: torch.dtype, gate: Optional[torch.Tensor] = None,
-                    out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """fp32 [T, C] in ``groups`` equal parts, each divided by its own root mean square, times weight; with ``gate`` [T, C] (a column view is
-    fine) also times ``sigmoid(gate)``, then times ``out_scale`` (csrc/kernels/residual_f32.cu).  ``out``: a [T, C] view with unit column
-    stride to write into (e.g. columns of a wider buffer)."""
-    if _use_native(x) and x.dtype == torch.float32 and x.is_contiguous() and out_dtype in (torch.bfloat16, torch.float32) and weight.dtype == out_dtype \
+def grouped_rmsnorm(x: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps: float, out_dtype: torch.dtype, gate: Optional[torch.Tensor] = None,
+                    out_scale: float = 1.0, out: Optional[torch.Tensor] = None, gate_act: str = "sigmoid") -> torch.Tensor:
+    """fp32 [T, C] in ``groups`` equal parts, each divided by its own root mean square, times weight (None: no weight); with ``gate`` [T, C] (a
+    column view is fine) also times ``sigmoid(gate)`` or ``silu(gate)`` (``gate_act``), then times ``out_scale`` (csrc/kernels/residual_f32.cu).
+    ``out``: a [T, C] view with unit column stride to write into (e.g. columns of a wider buffer)."""
+    if _use_native(x) and x.dtype == torch.float32 and x.is_contiguous() and out_dtype in (torch.bfloat16, torch.float32) \
+            and (weight is None or weight.dtype == out_dtype) \
             and x.shape[1] % groups == 0 and (gate is None or (gate.dtype == out_dtype and gate.stride(1) == 1)):
         if out is None:
             out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
         assert out.dtype == out_dtype and out.stride(1) == 1
-        torch.ops.sglb.grouped_rmsnorm(x, weight, int(groups), float(eps), out, gate, float(out_scale))
+        torch.ops.sglb.grouped_rmsnorm(x, weight, int(groups), float(eps), out, gate, float(out_scale), gate_act == "silu")
         return out
-    y = torch_ref.grouped_rmsnorm(x, weight, groups, eps, out_dtype, gate, out_scale)
+    y = torch_ref.grouped_rmsnorm(x, weight, groups, eps, out_dtype, gate, out_scale, gate_act)
     if out is not None:
         out.copy_(y)
         return out
@@ -688,10 +690,10 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
 def attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, positions: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       out_cache_loc: torch.Tensor, q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
                       inv_freq: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0, pad: int = 0,
-                      v_inv_freq: Optional[torch.Tensor] = None, v_interleaved: bool = False) -> torch.Tensor:
+                      v_inv_freq: Optional[torch.Tensor] = None, v_interleaved: bool = False, interleaved: bool = False) -> torch.Tensor:
     """what lies between the q / k / v projection and the attention kernel, in one pass per token: an RMS norm of q and of k over their whole
-    projection with a weight, a rotation of the first coordinates of every head by position (pairs half a rotary width apart, angles in
-    fp32 from ``inv_freq``), a blend of v with another layer's values of the same token, and the write of k / v rows into the paged cache
+    projection with a weight, a rotation of the first coordinates of every head by position (pairs half a rotary width apart, or neighbours with
+    ``interleaved``; angles in fp32 from ``inv_freq``), a blend of v with another layer's values of the same token, and the write of k / v rows into the paged cache
     (csrc/kernels/window_attention.cu; semantics in ``torch_ref.attention_prepare``).  ``qkv`` may be the first columns of a wider
     projection; ``v_first`` may be a column view.  ``v_inv_freq`` fp32 [Dv/2]: every value head is also turned over its whole width by
     ``position * v_inv_freq[m]`` before it is cached (pairs half a head apart, or neighbours with ``v_interleaved``).  Returns q [T, H, D | pad]
@@ -702,10 +704,10 @@ def attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, positi
             and (q_norm_w is None or (q_norm_w.dtype == qkv.dtype and k_norm_w.dtype == qkv.dtype))):
         q = torch.empty(qkv.shape[0], H, pad if pad > 0 else D, dtype=qkv.dtype, device=qkv.device)
         torch.ops.sglb.attention_prepare(qkv, int(H), int(G), int(D), int(Dv), positions, k_cache, v_cache, out_cache_loc, q_norm_w, k_norm_w, float(eps),
-                                         inv_freq, v_first, float(v_lambda), q, int(pad), v_inv_freq, bool(v_interleaved))
+                                         inv_freq, v_first, float(v_lambda), q, int(pad), v_inv_freq, bool(v_interleaved), bool(interleaved))
         return q
     return torch_ref.attention_prepare(qkv, H, G, D, Dv, positions, k_cache, v_cache, out_cache_loc, q_norm_w, k_norm_w, eps, inv_freq, v_first, v_lambda, pad,
-                                       v_inv_freq, v_interleaved)
+                                       v_inv_freq, v_interleaved, interleaved)
 
 
 def mamba1_scan(u: torch.Tensor, dt_raw: torch.Tensor, dt_bias: Optional[torch.Tensor], A_log: torch.Tensor, Bm: torch.Tensor, Cm: torch.Tensor,
@@ -897,3 +899,66 @@ def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     if x.is_cuda and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
         return torch.mm(x, w.t(), out_dtype=torch.float32)
     return torch.nn.functional.linear(x.float(), w.float())
+
+
+# ------------------------------------------------------------------ parallel residual streams / retention inputs / real-gated linear recurrence
+def stream_mix_norm(x: Optional[torch.Tensor], y: Optional[torch.Tensor], coef: torch.Tensor, streams: int, weight: torch.Tensor, eps: float,
+                    out_dtype: torch.dtype, centre: bool = True, table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, keep: bool = True):
+    """S parallel fp32 residual streams ``x`` [T, S, W] (in place): mix them, add a sublayer's output ``y`` to each, form the next sublayer's input
+    as a weighted sum of the new streams and norm it (layer norm without bias, or RMS norm), one kernel (csrc/kernels/streams.cu; semantics
+    and the packing of ``coef`` in ``torch_ref.stream_mix_norm``).  ``x`` None: every stream is the embedding row ``table[ids]`` (int32 ids).
+    ``keep`` False: the new streams are not stored.  Returns (streams | None, normed input in ``out_dtype``)."""
+    ref = x if x is not None else table
+    if (_use_native(ref) and coef.dtype == torch.float32 and streams <= 16 and weight.dtype == out_dtype and out_dtype in (torch.bfloat16, torch.float32)
+            and (x is None or (x.dtype == torch.float32 and x.is_contiguous())) and (y is None or (y.dtype == out_dtype and y.is_contiguous()))
+            and (table is None or (table.dtype in (torch.bfloat16, torch.float32) and table.is_contiguous()))):
+        T, W = (ids.shape[0], table.shape[1]) if x is None else (x.shape[0], x.shape[2])
+        h = torch.empty(T, W, dtype=out_dtype, device=ref.device)
+        new = None if not keep else x if x is not None else torch.empty(T, streams, W, dtype=torch.float32, device=ref.device)
+        torch.ops.sglb.stream_mix_norm(x, table if x is None else None, ids.int() if x is None else None, y, coef, int(streams), weight, float(eps), bool(centre),
+                                       new if (y is not None or x is None) else None, h)
+        return new, h
+    return torch_ref.stream_mix_norm(x, y, coef, streams, weight, eps, out_dtype, centre, table, ids, keep)
+
+
+def linear_attention_prepare(proj: torch.Tensor, H: int, D: int, Dv: int, positions: torch.Tensor, inv_freq: Optional[torch.Tensor] = None,
+                             interleaved: bool = False, k_scale: float = 1.0, silu: bool = False) -> torch.Tensor:
+    """projection rows [v | k | q | ...] -> the fp32 scan input [v | k | q] of linear attention: optional SiLU, rotation of the first coordinates
+    of every k and q head by position (fp32 angles), a constant on k (csrc/kernels/mamba.cu; semantics in ``torch_ref.linear_attention_prepare``)"""
+    if _use_native(proj) and proj.dtype in (torch.bfloat16, torch.float32) and proj.stride(1) == 1:
+        u = torch.empty(proj.shape[0], H * (Dv + 2 * D), dtype=torch.float32, device=proj.device)
+        torch.ops.sglb.linear_attention_prepare(proj, int(H), int(D), int(Dv), positions, inv_freq, bool(interleaved), float(k_scale), bool(silu), u)
+        return u
+    return torch_ref.linear_attention_prepare(proj, H, D, Dv, positions, inv_freq, interleaved, k_scale, silu)
+
+
+DIAG_TC = True          # the tcgen05 route of block_linear_f32 (tests compare it with the general one)
+
+
+def block_linear_f32(u: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """block-diagonal product with an fp32 result: u [T, blocks * n], w [blocks, m, n] -> [T, blocks, m].  bf16: the tcgen05 GEMM with a column offset
+    per block (csrc/kernels/gemm_tc.cu; n a multiple of 8, m of 32); fp32 serving and other sizes: fp32 products per block"""
+    nb, m, n = w.shape
+    if (DIAG_TC and _use_native(u) and u.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and u.stride(1) == 1 and u.stride(0) % 8 == 0
+            and u.data_ptr() % 16 == 0 and n % 8 == 0 and m % 32 == 0 and w.is_contiguous()):
+        out = torch.empty(u.shape[0], nb, m, dtype=torch.float32, device=u.device)
+        torch.ops.sglb.gemm_diag_f32(u, w, out)
+        return out
+    return torch_ref.block_linear_f32(u, w).contiguous()
+
+
+def rglru_scan(gates: torch.Tensor, gate_bias: Optional[torch.Tensor], u: torch.Tensor, lam: torch.Tensor, y: torch.Tensor, state: torch.Tensor,
+               req_slots: torch.Tensor, seq_lens: torch.Tensor, cu_q: Optional[torch.Tensor], q_lens: Optional[torch.Tensor], blocks: int,
+               power: float = 8.0) -> torch.Tensor:
+    """real-gated linear recurrent unit over a ragged batch (prompt portions and decode tokens alike): gate activations, decay, the fp32 recurrence
+    ``S <- a S + sqrt(1 - a^2) i u`` with ``log a = -power r softplus(lam)`` and the product with ``gelu_tanh(y)`` in one kernel
+    (csrc/kernels/rglru.cu; semantics in ``torch_ref.rglru_scan``).  ``gates`` fp32 [T, blocks, 2 C / blocks] from ``block_linear_f32``; ``u`` and
+    ``y`` (a column view is fine) in the model dtype, which is also the result's."""
+    T, C = u.shape
+    if (_use_native(u) and u.dtype in (torch.bfloat16, torch.float32) and u.stride(1) == 1 and y.dtype == u.dtype and y.stride(1) == 1
+            and gates.dtype == torch.float32 and gates.is_contiguous() and state.dtype == torch.float32 and state.is_contiguous()
+            and lam.dtype == torch.float32 and req_slots.numel() <= 65535 and (gate_bias is None or (gate_bias.dtype == torch.float32 and gate_bias.is_contiguous()))):
+        out = torch.empty(T, C, dtype=u.dtype, device=u.device)
+        torch.ops.sglb.rglru_scan(gates, gate_bias, u, lam, y, state, req_slots, seq_lens, cu_q, int(blocks), float(power), out)
+        return out
+    return torch_ref.rglru_scan(gates, gate_bias, u, lam, y, state, req_slots, seq_lens, q_lens, u.dtype, blocks, power)

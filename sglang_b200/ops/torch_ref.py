@@ -524,15 +524,17 @@ def postnorm_add_rmsnorm_f32(residual: torch.Tensor, delta: Optional[torch.Tenso
     return (y * g(weight)).to(out_dtype)
 
 
-def grouped_rmsnorm(x: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, out_dtype: torch.dtype, gate: Optional[torch.Tensor] = None,
-                    out_scale: float = 1.0) -> torch.Tensor:
-    """x [T, C] cut into ``groups`` equal parts, each divided by its own root mean square, times weight [C]; with ``gate`` [T, C] also times
-    ``sigmoid(gate)``; times ``out_scale``"""
+def grouped_rmsnorm(x: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps: float, out_dtype: torch.dtype, gate: Optional[torch.Tensor] = None,
+                    out_scale: float = 1.0, gate_act: str = "sigmoid") -> torch.Tensor:
+    """x [T, C] cut into ``groups`` equal parts, each divided by its own root mean square, times weight [C] (if any); with ``gate`` [T, C] also
+    times ``sigmoid(gate)`` or ``silu(gate)``; times ``out_scale``"""
     T, C = x.shape
     xf = x.float().view(T, groups, C // groups)
-    y = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)).view(T, C) * weight.float()
+    y = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)).view(T, C)
+    if weight is not None:
+        y = y * weight.float()
     if gate is not None:
-        y = y * torch.sigmoid(gate.float())
+        y = y * (F.silu(gate.float()) if gate_act == "silu" else torch.sigmoid(gate.float()))
     return (y * out_scale if out_scale != 1.0 else y).to(out_dtype)
 
 
@@ -757,13 +759,13 @@ def conv_attention_prepare(qkv: torch.Tensor, H: int, G: int, M: int, D: int, Dv
 def attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, positions: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       out_cache_loc: torch.Tensor, q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
                       inv_freq: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0, pad: int = 0,
-                      v_inv_freq: Optional[torch.Tensor] = None, v_interleaved: bool = False) -> torch.Tensor:
+                      v_inv_freq: Optional[torch.Tensor] = None, v_interleaved: bool = False, interleaved: bool = False) -> torch.Tensor:
     """rows of ``qkv`` [T, >= H*D + G*D + G*Dv] = [q | k | v | ...] -> q [T, H, D] in the cache dtype; k rows to ``k_cache[loc]`` (first
     ``G*D`` columns), v rows to ``v_cache[loc]`` (first ``G*Dv`` columns).  In this order:
 
     * ``q_norm_w`` [H*D] / ``k_norm_w`` [G*D]: q and k are RMS-normed over their WHOLE projection (all heads at once), times the weight;
-    * ``inv_freq`` fp32 [R/2]: the first R coordinates of every q and k head are rotated by the angle ``position * inv_freq[i]``, coordinate
-      ``i`` paired with ``i + R/2``;
+    * ``inv_freq`` fp32 [R/2]: the first R coordinates of every q and k head are rotated by the angle ``position * inv_freq[i]``, pair i =
+      coordinates ``(i, i + R/2)``, or ``(2i, 2i + 1)`` with ``interleaved``;
     * ``v_first`` [T, G*Dv]: v <- (1 - v_lambda) v + v_lambda v_first before it is cached;
     * ``v_inv_freq`` fp32 [Dv/2]: every value head is rotated over its whole width by ``position * v_inv_freq[m]`` before it is cached, pair m
       = coordinates ``(m, m + Dv/2)``, or ``(2m, 2m + 1)`` with ``v_interleaved`` (``rotate_heads`` turns an attention output back).
@@ -778,15 +780,7 @@ def attention_prepare(qkv: torch.Tensor, H: int, G: int, D: int, Dv: int, positi
         k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * k_norm_w.float()
     q, k = q.reshape(T, H, D), k.reshape(T, G, D)
     if inv_freq is not None:
-        half = inv_freq.numel()
-        ang = positions.float()[:, None] * inv_freq.float()[None, :]
-        c, s = torch.cos(ang)[:, None, :], torch.sin(ang)[:, None, :]
-
-        def rot(x):
-            a, b = x[..., :half], x[..., half:2 * half]
-            return torch.cat([a * c - b * s, b * c + a * s, x[..., 2 * half:]], -1)
-
-        q, k = rot(q), rot(k)
+        q, k = rotate_pairs(q, positions, inv_freq, interleaved), rotate_pairs(k, positions, inv_freq, interleaved)
     if v_first is not None:
         v = (1.0 - v_lambda) * v + v_lambda * v_first.float()
     if v_inv_freq is not None:
@@ -982,3 +976,79 @@ def mamba1_scan(u: torch.Tensor, dt_raw: torch.Tensor, dt_bias: Optional[torch.T
     if z is not None:
         out = out * F.silu(z.float())
     return out.to(out_dtype)
+
+
+def linear_attention_prepare(proj: torch.Tensor, H: int, D: int, Dv: int, positions: torch.Tensor, inv_freq: Optional[torch.Tensor], interleaved: bool,
+                             k_scale: float, silu: bool) -> torch.Tensor:
+    """projection rows [v (H*Dv) | k (H*D) | q (H*D) | ...] -> the same columns in fp32, the scan's [x | B | C]: ``silu`` of everything (if asked),
+    the first ``2 * len(inv_freq)`` coordinates of every k and q head turned by ``position * inv_freq[m]`` (``rotate_pairs``), k times ``k_scale``"""
+    T, nv, nk = proj.shape[0], H * Dv, H * D
+    u = proj[:, :nv + 2 * nk].float()
+    if silu:
+        u = F.silu(u)
+    v, k, q = u[:, :nv], u[:, nv:nv + nk].reshape(T, H, D), u[:, nv + nk:].reshape(T, H, D)
+    if inv_freq is not None:
+        k, q = rotate_pairs(k, positions, inv_freq, interleaved), rotate_pairs(q, positions, inv_freq, interleaved)
+    return torch.cat([v, (k * k_scale).reshape(T, nk), q.reshape(T, nk)], 1).contiguous()
+
+
+def stream_mix_norm(x: Optional[torch.Tensor], y: Optional[torch.Tensor], coef: torch.Tensor, streams: int, weight: torch.Tensor, eps: float,
+                    out_dtype: torch.dtype, centre: bool, table: Optional[torch.Tensor], ids: Optional[torch.Tensor], keep: bool):
+    """parallel residual streams x fp32 [T, S, W] (None: all equal to the rows ``table[ids]``).  ``coef`` fp32 [S*S + 2*S] = mix [from, to] | out | in.
+    With ``y`` [T, W]: x'_t = sum_s mix[s, t] x_s + out[t] y (all from the old streams; without: x' = x).  u = sum_s in[s] x'_s, and
+    h = (u - mean) / sqrt(variance + eps) * weight (``centre``) or u / rms(u) * weight.  Returns (x' | None unless ``keep``, h in ``out_dtype``)"""
+    S = streams
+    mix, out, cin = coef[:S * S].view(S, S), coef[S * S:S * S + S], coef[S * S + S:]
+    old = x if x is not None else table[ids.long()].float()[:, None, :].expand(-1, S, -1)
+    new = old
+    if y is not None:
+        new = torch.einsum("tsw,sr->trw", old, mix) + out[None, :, None] * y.float()[:, None, :]
+    u = torch.einsum("tsw,s->tw", new, cin)
+    if centre:
+        u = u - u.mean(-1, keepdim=True)
+    h = (u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype)
+    if not keep:
+        return None, h
+    if x is None:
+        return new.contiguous(), h
+    if y is not None:
+        x.copy_(new)
+    return x, h
+
+
+def block_linear_f32(u: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """block-diagonal product with an fp32 result: u [T, blocks * n], w [blocks, m, n] -> [T, blocks, m]"""
+    nb, _, n = w.shape
+    return torch.einsum("tbn,bmn->tbm", u.float().view(-1, nb, n), w.float())
+
+
+def rglru_scan(gates: torch.Tensor, gate_bias: Optional[torch.Tensor], u: torch.Tensor, lam: torch.Tensor, y: torch.Tensor, state: torch.Tensor,
+               req_slots: torch.Tensor, seq_lens: torch.Tensor, q_lens: Optional[torch.Tensor], out_dtype: torch.dtype, blocks: int,
+               power: float = 8.0) -> torch.Tensor:
+    """real-gated linear recurrent unit over a ragged batch, token by token, state in place.
+
+    gates fp32 [T, blocks, 2, C / blocks] (recurrence gate, input gate before their sigmoids; ``gate_bias`` fp32 [blocks, 2, C / blocks] is added);
+    u [T, C]; lam fp32 [C]; y [T, C] the other branch.  r, i = sigmoid(gates + bias);  log a = -power r softplus(lam);  state fp32
+    [slots, 1, 1, C]:  S <- a S + sqrt(1 - a^2) i u;  returns S * gelu_tanh(y) in ``out_dtype``.  A request whose ``seq_len == q_len`` starts from zero."""
+    T, C = u.shape
+    g = gates.float().view(T, blocks, 2, C // blocks)
+    if gate_bias is not None:
+        g = g + gate_bias.float().view(1, blocks, 2, C // blocks)
+    r, i = torch.sigmoid(g[:, :, 0]).reshape(T, C), torch.sigmoid(g[:, :, 1]).reshape(T, C)
+    la = -power * r * F.softplus(lam.float())
+    a = torch.exp(la)
+    b = torch.sqrt(-torch.expm1(2.0 * la)) * i * u.float()
+    out = torch.empty(T, C, dtype=torch.float32, device=u.device)
+    off = 0
+    for k in range(req_slots.shape[0]):
+        n = 1 if q_lens is None else int(q_lens[k])
+        if n <= 0:
+            continue
+        slot = int(req_slots[k])
+        S = torch.zeros(C, dtype=torch.float32, device=u.device) if int(seq_lens[k]) - n == 0 else state[slot].reshape(C).clone()
+        for t in range(off, off + n):
+            S = a[t] * S + b[t]
+            out[t] = S
+        state[slot] = S.view(state.shape[1:])
+        off += n
+    return (out * F.gelu(y.float(), approximate="tanh")).to(out_dtype)
