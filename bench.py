@@ -50,10 +50,11 @@ def parse_args():
                     help="instead of the default workload: Rirotar beside Qwen3-Next at equal size (engine prefill / decode) and its kernels beside "
                          "the like ops, one JSON line per measurement (sglang_b200/benchmark/hybrid_compare.py)")
     ap.add_argument("--hybrid-sizes", default="2048,4096", help="model widths of --hybrid-compare")
-    ap.add_argument("--hybrid-family", default="rirotar", choices=("rirotar", "zaparax", "resatar", "rumuvik", "mumasun"),
+    ap.add_argument("--hybrid-family", default="rirotar", choices=("rirotar", "zaparax", "resatar", "rumuvik", "mumasun", "surasun"),
                     help="which per-layer hybrid family --hybrid-compare measures: rirotar beside Qwen3-Next, zaparax beside Nemotron-H "
                          "(sglang_b200/benchmark/zaparax_compare.py), resatar beside Jamba (sglang_b200/benchmark/resatar_compare.py), rumuvik beside "
-                         "Resatar (sglang_b200/benchmark/rumuvik_compare.py), or mumasun beside Qwen3-MoE (sglang_b200/benchmark/mumasun_compare.py)")
+                         "Resatar (sglang_b200/benchmark/rumuvik_compare.py), mumasun beside Qwen3-MoE (sglang_b200/benchmark/mumasun_compare.py), or surasun "
+                         "beside Resatar (sglang_b200/benchmark/surasun_compare.py)")
     return ap.parse_args()
 
 
@@ -208,6 +209,8 @@ def main() -> None:
             from sglang_b200.benchmark.rumuvik_compare import main as hybrid_main
         elif args.hybrid_family == "mumasun":
             from sglang_b200.benchmark.mumasun_compare import main as hybrid_main
+        elif args.hybrid_family == "surasun":
+            from sglang_b200.benchmark.surasun_compare import main as hybrid_main
         else:
             from sglang_b200.benchmark.hybrid_compare import main as hybrid_main
 

@@ -208,7 +208,7 @@ void causal_conv1d(const at::Tensor& x, const at::Tensor& w, c10::optional<at::T
   sglb::causal_conv1d(x.data_ptr(), (int)x.stride(0), w.data_ptr(), bias.has_value() ? bias->data_ptr() : nullptr, conv_state.data_ptr(),
                       opt_ptr<int>(cu_q), req_slots.data_ptr<int>(), seq_lens.data_ptr<int>(), (int)req_slots.size(0), (int)max_q_len, C, K, silu, bf16,
                       u.data_ptr(), u.scalar_type() == at::kBFloat16, (int)u.stride(0), cur_stream());
-  count(2);
+  count();
 }
 
 // Mamba-2 decode: S = S * exp(dt A) + dt x B ; y = <S, C> + D x   (state fp32 [slots, H, P, N], one token per request)

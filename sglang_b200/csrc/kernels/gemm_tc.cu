@@ -53,11 +53,13 @@ struct GemmCfg {
   static constexpr int STAGES = (BN >= 256) ? 4 : (BN >= 128 ? 6 : 8);
   static constexpr int TMEM_COLS = (2 * BN < 32) ? 32 : 2 * BN;
   static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 /*align slack*/ + 256 /*barriers*/;
+  static constexpr int OUT_BYTES = 4 * 2 * 4096;      // EPI_F32_DIAG: two 32 x 32 fp32 staging tiles per epilogue warp, behind the barriers
+  static constexpr int SMEM_BYTES_F32 = STAGES * STAGE_BYTES + 1024 + 1024 + OUT_BYTES;
 };
 
 template <int BN, int EPI, bool GROUPED>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
-gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
+gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const __grid_constant__ CUtensorMap tmC,
                __nv_bfloat16* __restrict__ C, const __nv_bfloat16* __restrict__ bias, int M, int N, int K, int ldc,
                const GemmPush push, const int* __restrict__ tile_expert, const int* __restrict__ num_m_tiles_ptr, int n_half) {
   constexpr bool SPLIT = (EPI == EPI_SILU_SPLIT);
@@ -150,6 +152,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
   } else if (warp >= 4) {
     // ------------------------------------------------------------ epilogue
     const int q = warp - 4;  // == warp % 4 : TMEM lane quadrant this warp may access
+    [[maybe_unused]] uint8_t* sOut = smem + STAGES * Cfg::STAGE_BYTES + 1024 + q * 2 * 4096;
+    [[maybe_unused]] int out_buf = 0;
     int acc = 0; uint32_t acc_phase = 0;
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x) {
       const int m_blk = tile % m_tiles, n_blk = tile / m_tiles;
@@ -187,6 +191,23 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         }
         tmem_ld_wait();
         const int col0 = n_blk * BN + c * 32;
+        if constexpr (EPI == EPI_F32_DIAG) {
+          // 32 rows x 32 columns through shared memory (128-byte rows, 128-byte swizzle) and out by TMA: rows beyond M are clipped by the map
+          uint8_t* buf = sOut + out_buf * 4096;
+          if (lane == 0) tma_store_wait_read1();          // the store that read this buffer two chunks ago is done with it
+          __syncwarp();
+#pragma unroll
+          for (int v = 0; v < 8; ++v)
+            *reinterpret_cast<uint4*>(buf + lane * 128 + ((v ^ (lane & 7)) << 4)) = make_uint4(r[4 * v], r[4 * v + 1], r[4 * v + 2], r[4 * v + 3]);
+          fence_proxy_async_smem();
+          __syncwarp();
+          if (lane == 0 && col0 < N) {
+            tma_store_2d(&tmC, buf, col0, m_blk * GEMM_BM + q * 32);
+            tma_store_commit();
+          }
+          out_buf ^= 1;
+          continue;
+        }
         if (EPI == EPI_SILU_MUL) {
           // columns [0,16) = gate, [16,32) = up of the same 16 intermediate features
           if (row < M && col0 < N) {
@@ -212,12 +233,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 float f[8];
 #pragma unroll
                 for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(r[v * 8 + i]);
-                if (EPI == EPI_F32_DIAG) {
-                  float* dst = reinterpret_cast<float*>(C) + (size_t)row * ldc + col;
-                  *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
-                  *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
-                  continue;
-                }
                 if (EPI == EPI_ROWSCALE) {
 #pragma unroll
                   for (int i = 0; i < 8; ++i) f[i] *= row_scale;
@@ -249,6 +264,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       __syncwarp();
       if (lane == 0) mbar_arrive(&tempty[acc]);
       if (++acc == 2) { acc = 0; acc_phase ^= 1; }
+    }
+    if constexpr (EPI == EPI_F32_DIAG) {
+      if (lane == 0) tma_store_wait0();
     }
   }
 
@@ -304,15 +322,22 @@ static void launch_gemm(const void* A, const void* W, void* C, const void* bias,
     uint32_t bB[2] = {GEMM_BK, (uint32_t)BN_OUT};
     tmB = make_tmap(W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dB, sBs, bB, CU_TENSOR_MAP_SWIZZLE_128B);
   }
+  constexpr int smem = EPI == EPI_F32_DIAG ? Cfg::SMEM_BYTES_F32 : Cfg::SMEM_BYTES;
+  CUtensorMap tmC = tmA;
+  if (EPI == EPI_F32_DIAG) {
+    uint64_t dC[2] = {(uint64_t)N, (uint64_t)M}, sC[1] = {(uint64_t)ldc * 4};
+    uint32_t bC[2] = {32, 32};
+    tmC = make_tmap(C, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 2, dC, sC, bC, CU_TENSOR_MAP_SWIZZLE_128B);
+  }
   auto kern = gemm_tc_kernel<BN, EPI, GROUPED>;
   static bool configured = false;
   if (!configured) {
-    SGLB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
+    SGLB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     configured = true;
   }
   const int m_tiles = (M + GEMM_BM - 1) / GEMM_BM, n_tiles = (N + BN_OUT - 1) / BN_OUT;
   const int grid = (int)std::min<long long>((long long)m_tiles * n_tiles, num_sms);
-  kern<<<grid, GEMM_THREADS, Cfg::SMEM_BYTES, stream>>>(tmA, tmB, (__nv_bfloat16*)C, (const __nv_bfloat16*)bias, M, N, K, ldc, push,
+  kern<<<grid, GEMM_THREADS, smem, stream>>>(tmA, tmB, tmC, (__nv_bfloat16*)C, (const __nv_bfloat16*)bias, M, N, K, ldc, push,
                                                         ex.tile_expert, ex.num_m_tiles, ex.n_half);
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
@@ -382,10 +407,10 @@ void gemm_bf16_tc_diag_f32(const void* A, const void* W, float* C, int M, int bl
   GemmExtra ex; ex.n_half = rows; ex.a_cols = blocks * K;
   const int N = blocks * rows, m_tiles = (M + GEMM_BM - 1) / GEMM_BM;
   int bn = 32;
-  for (int cand : {128, 64, 32}) {
+  for (int cand : {256, 128, 64, 32}) {
     if (rows % cand) continue;
     bn = cand;
-    if ((long long)m_tiles * (N / cand) >= num_sms) break;
+    if ((long long)m_tiles * (N / cand) >= 2LL * num_sms) break;
   }
   dispatch_bn<EPI_F32_DIAG>(bn, A, W, C, nullptr, M, N, K, lda, K, N, num_sms, stream, GemmPush{}, ex);
 }

@@ -1,7 +1,7 @@
 // State-space (Mamba / Mamba-2) kernels: causal depthwise conv1d over ragged batches with a per-request rolling state, and the
 // single-token selective state update of decode.
 //
-//   causal_conv1d (prefill / extend / decode):  u[t, c] = act(bias[c] + sum_{j<k} w[c, j] * x[t - (k-1) + j, c]),   x[<0] taken from conv_state
+//   causal_conv1d (prefill / extend / decode, one launch):  u[t, c] = act(bias[c] + sum_{j<k} w[c, j] * x[t - (k-1) + j, c]),   x[<0] taken from conv_state
 //        conv_state[slot, c, :] <- the last k-1 inputs of the request (shifted by the new tokens)
 //   selective_state_update (decode):            S[b,h,p,:] = S * exp(dt[b,h] * A[h]) + dt[b,h] * x[b,h,p] * B[b,g,:]
 //                                               y[b,h,p]   = <S[b,h,p,:], C[b,g,:]> + D[h] * x[b,h,p]
@@ -19,7 +19,7 @@
 namespace sglb {
 
 constexpr int CONV_MAX_K = 8;
-constexpr int CONV_CHUNK = 128;      // tokens per block along a request
+constexpr int CONV_CHUNK = 64;       // tokens per block along a request (more than any number of taps)
 
 template <typename T> __device__ __forceinline__ float ld_f(const T* p);
 template <> __device__ __forceinline__ float ld_f<float>(const float* p) { return *p; }
@@ -28,13 +28,31 @@ template <typename T> __device__ __forceinline__ void st_f(T* p, float v);
 template <> __device__ __forceinline__ void st_f<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void st_f<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
-// grid (ceil(C / 256), chunks, B); thread = channel.  cu_q == nullptr: decode (one token per request, row = request index).
-template <typename T, typename TU>
-__global__ void __launch_bounds__(256) causal_conv1d_fwd_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, const T* __restrict__ bias,
-                                                                const T* __restrict__ conv_state, const int* __restrict__ cu_q,
-                                                                const int* __restrict__ req_slots, const int* __restrict__ seq_lens, int C, int K,
-                                                                int silu, TU* __restrict__ u, int ldu) {
-  const int c = blockIdx.x * 256 + threadIdx.x;
+// grid (ceil(C / (256 VEC)), chunks, B); a thread owns VEC neighbouring channels and walks a chunk of tokens, CONV_RUN rows loaded at a time, one
+// run ahead.  cu_q == nullptr: decode (one token per request, row = request index).  Only a request's first chunk looks back beyond this call's
+// tokens, so its threads also roll the state forward by the call's tokens (they have read the old columns by then; nobody else touches them).
+// KT: taps at compile time (0: at run time, 2..8).
+template <typename T> __device__ __forceinline__ void conv_ld2(const T* p, float* v);
+template <> __device__ __forceinline__ void conv_ld2<float>(const float* p, float* v) {
+  const float2 w = *reinterpret_cast<const float2*>(p);
+  v[0] = w.x; v[1] = w.y;
+}
+template <> __device__ __forceinline__ void conv_ld2<__nv_bfloat16>(const __nv_bfloat16* p, float* v) {
+  const uint32_t w = *reinterpret_cast<const uint32_t*>(p);
+  v[0] = bf16_lo(w); v[1] = bf16_hi(w);
+}
+__device__ __forceinline__ void conv_st2(float* p, const float* v) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); }
+__device__ __forceinline__ void conv_st2(__nv_bfloat16* p, const float* v) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(v[0], v[1]); }
+
+constexpr int CONV_RUN = 8;
+
+template <typename T, typename TU, int KT, int VEC>
+__global__ void __launch_bounds__(256) causal_conv1d_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, const T* __restrict__ bias,
+                                                            T* __restrict__ conv_state, const int* __restrict__ cu_q, const int* __restrict__ req_slots,
+                                                            const int* __restrict__ seq_lens, int C, int Kr, int silu, TU* __restrict__ u, int ldu) {
+  constexpr int KM = KT > 0 ? KT : CONV_MAX_K;
+  const int K = KT > 0 ? KT : Kr;
+  const int c = (blockIdx.x * 256 + threadIdx.x) * VEC;
   const int b = blockIdx.z;
   if (c >= C) return;
   const int q0 = cu_q ? cu_q[b] : b;
@@ -43,68 +61,105 @@ __global__ void __launch_bounds__(256) causal_conv1d_fwd_kernel(const T* __restr
   if (t0 >= n) return;
   const int t1 = min(n, t0 + CONV_CHUNK);
   const bool fresh = seq_lens[b] - n == 0;            // first tokens of the request: the state is all zeros, whatever the slot holds
-  const T* st = conv_state + ((size_t)req_slots[b] * C + c) * (K - 1);
-  float wk[CONV_MAX_K], win[CONV_MAX_K];
+  T* st = conv_state + ((size_t)req_slots[b] * C + c) * (K - 1);
+  const T* xr = x + (size_t)q0 * ldx + c;
+  auto load = [&](int t, float* v) {
+    const T* p = xr + (size_t)t * ldx;
+    if constexpr (VEC == 2) conv_ld2<T>(p, v);
+    else v[0] = ld_f<T>(p);
+  };
+  float nx[CONV_RUN][VEC];                             // the next run's rows: they fly while the current run is computed
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_K; ++j) wk[j] = j < K ? ld_f<T>(w + (size_t)c * K + j) : 0.f;
-  const float bs = bias ? ld_f<T>(bias + c) : 0.f;
-  float w_last = 0.f;
+  for (int k = 0; k < CONV_RUN; ++k) load(min(t0 + k, t1 - 1), nx[k]);
+  float wk[VEC][KM], win[VEC][KM], bs[VEC];           // win: the K - 1 inputs before the current token, oldest first
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_K; ++j)
-    if (j == K - 1) w_last = wk[j];
+  for (int e = 0; e < VEC; ++e) {
+#pragma unroll
+    for (int j = 0; j < KM; ++j) wk[e][j] = j < K ? ld_f<T>(w + (size_t)(c + e) * K + j) : 0.f;
+    bs[e] = bias ? ld_f<T>(bias + c + e) : 0.f;
+  }
   // window = inputs t0-(K-1) .. t0-1: from x when inside this call's tokens, else from the rolling state (position relative to its end)
+  float old[VEC][KM];                                  // the state's columns, where this chunk looks at them
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_K - 1; ++j) {
+  for (int j = 0; j < KM - 1; ++j) {
     if (j < K - 1) {
       const int t = t0 - (K - 1) + j;
-      float v = 0.f;
-      if (t >= 0) v = ld_f<T>(x + (size_t)(q0 + t) * ldx + c);
-      else if (!fresh) v = ld_f<T>(st + (K - 1) + t);
-      win[j] = v;
+      float v[VEC];
+      if (t >= 0) load(t, v);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        old[e][j] = 0.f;
+        if (t < 0) {                                   // then t0 == 0: column (K - 1) + t = j
+          v[e] = fresh ? 0.f : ld_f<T>(st + (size_t)e * (K - 1) + j);
+          old[e][j] = v[e];
+        }
+        win[e][j] = v[e];
+      }
     }
   }
-  for (int t = t0; t < t1; ++t) {
-    const float xv = ld_f<T>(x + (size_t)(q0 + t) * ldx + c);
-    float acc = bs + w_last * xv;
+  for (int r0 = t0; r0 < t1; r0 += CONV_RUN) {
+    float xs[CONV_RUN][VEC];
 #pragma unroll
-    for (int j = 0; j < CONV_MAX_K - 1; ++j)
-      if (j < K - 1) acc += wk[j] * win[j];
+    for (int k = 0; k < CONV_RUN; ++k)
 #pragma unroll
-    for (int j = 0; j < CONV_MAX_K - 1; ++j) {
-      if (j < K - 2) win[j] = win[j + 1];
-      else if (j == K - 2) win[j] = xv;
+      for (int e = 0; e < VEC; ++e) xs[k][e] = nx[k][e];
+    if (r0 + CONV_RUN < t1) {
+#pragma unroll
+      for (int k = 0; k < CONV_RUN; ++k) load(min(r0 + CONV_RUN + k, t1 - 1), nx[k]);
     }
-    if (silu) acc = acc / (1.f + __expf(-acc));
-    st_f<TU>(u + (size_t)(q0 + t) * ldu + c, acc);
-  }
-}
-
-// second pass (stream-ordered after the forward, which still reads the OLD state): roll the state forward by the request's new tokens
-template <typename T>
-__global__ void __launch_bounds__(256) causal_conv1d_state_kernel(const T* __restrict__ x, int ldx, T* __restrict__ conv_state, const int* __restrict__ cu_q,
-                                                                  const int* __restrict__ req_slots, const int* __restrict__ seq_lens, int C, int K) {
-  const int c = blockIdx.x * 256 + threadIdx.x;
-  const int b = blockIdx.y;
-  if (c >= C) return;
-  const int q0 = cu_q ? cu_q[b] : b;
-  const int n = cu_q ? cu_q[b + 1] - q0 : 1;
-  if (n <= 0) return;
-  const bool fresh = seq_lens[b] - n == 0;
-  T* st = conv_state + ((size_t)req_slots[b] * C + c) * (K - 1);
-  float nw[CONV_MAX_K];
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_K - 1; ++j) {
-    if (j < K - 1) {
-      const int t = n - (K - 1) + j;                 // input index (relative to this call) that ends up in state column j
-      float v = 0.f;
-      if (t >= 0) v = ld_f<T>(x + (size_t)(q0 + t) * ldx + c);
-      else if (!fresh) v = ld_f<T>(st + (K - 1) + t);
-      nw[j] = v;
+    for (int k = 0; k < CONV_RUN; ++k) {
+      if (r0 + k >= t1) break;
+      float acc[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        float wl = wk[e][KM - 1];
+        if (KT == 0) {
+#pragma unroll
+          for (int j = 0; j < KM; ++j)
+            if (j == K - 1) wl = wk[e][j];
+        }
+        float a = bs[e] + wl * xs[k][e];
+#pragma unroll
+        for (int j = 0; j < KM - 1; ++j)
+          if (j < K - 1) a += wk[e][j] * win[e][j];
+#pragma unroll
+        for (int j = 0; j < KM - 1; ++j) {
+          if (j < K - 2) win[e][j] = win[e][j + 1];
+          else if (j == K - 2) win[e][j] = xs[k][e];
+        }
+        if (silu) a = a / (1.f + __expf(-a));
+        acc[e] = a;
+      }
+      TU* dst = u + (size_t)(q0 + r0 + k) * ldu + c;
+      if constexpr (VEC == 2) conv_st2(dst, acc);
+      else st_f<TU>(dst, acc[0]);
     }
   }
+  if (t0 == 0) {                                       // roll the state: column j takes input n - (K - 1) + j
+    float nw[KM][VEC];
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_K - 1; ++j)
-    if (j < K - 1) st_f<T>(st + j, nw[j]);
+    for (int j = 0; j < KM - 1; ++j) {
+      if (j < K - 1) {
+        const int t = n - (K - 1) + j;
+        if (t >= 0) load(t, nw[j]);
+        else {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            nw[j][e] = 0.f;
+#pragma unroll
+            for (int i = 0; i < KM - 1; ++i)
+              if (i == (K - 1) + t) nw[j][e] = old[e][i];
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e)
+#pragma unroll
+      for (int j = 0; j < KM - 1; ++j)
+        if (j < K - 1) st_f<T>(st + (size_t)e * (K - 1) + j, nw[j][e]);
+  }
 }
 
 // the state half alone, for kernels that convolve on their own (any number of taps: columns are moved one by one, oldest first)
@@ -137,27 +192,34 @@ void causal_conv1d_state(const void* x, int ldx, void* conv_state, const int* cu
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
 
+template <typename T, typename TU>
+void dispatch_conv1d(const void* x, int ldx, const void* w, const void* bias, void* conv_state, const int* cu_q, const int* req_slots, const int* seq_lens,
+                     int B, int max_q_len, int C, int K, bool silu, void* u, int ldu, cudaStream_t stream) {
+  const int chunks = (std::max(max_q_len, 1) + CONV_CHUNK - 1) / CONV_CHUNK;
+  const bool two = C % 2 == 0 && ldx % 2 == 0 && ldu % 2 == 0 && (uintptr_t)x % (2 * sizeof(T)) == 0 && (uintptr_t)u % (2 * sizeof(TU)) == 0 &&
+                   (long long)((C + 511) / 512) * chunks * B >= 296;          // enough CTAs with two channels per thread
+  dim3 grid((C + (two ? 511 : 255)) / (two ? 512 : 256), chunks, B);
+#define SGLB_CONV(KT, VEC)                                                                                                                            \
+  causal_conv1d_kernel<T, TU, KT, VEC><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, (const T*)bias, (T*)conv_state, cu_q, req_slots, seq_lens, \
+                                                                 C, K, silu ? 1 : 0, (TU*)u, ldu)
+  if (K == 4) { if (two) SGLB_CONV(4, 2); else SGLB_CONV(4, 1); }
+  else if (K == 3) { if (two) SGLB_CONV(3, 2); else SGLB_CONV(3, 1); }
+  else if (K == 2) { if (two) SGLB_CONV(2, 2); else SGLB_CONV(2, 1); }
+  else { if (two) SGLB_CONV(0, 2); else SGLB_CONV(0, 1); }
+#undef SGLB_CONV
+  SGLB_CUDA_CHECK(cudaGetLastError());
+}
+
 void causal_conv1d(const void* x, int ldx, const void* w, const void* bias, void* conv_state, const int* cu_q, const int* req_slots,
                    const int* seq_lens, int B, int max_q_len, int C, int K, bool silu, bool bf16, void* u, bool u_bf16, int ldu, cudaStream_t stream) {
   if (B <= 0) return;
   if (K < 2 || K > CONV_MAX_K) throw std::runtime_error("sglb causal_conv1d: kernel width must be 2..8");
   if (u_bf16 && !bf16) throw std::runtime_error("sglb causal_conv1d: the output is fp32 or of the input's type");
-  dim3 g1((C + 255) / 256, (std::max(max_q_len, 1) + CONV_CHUNK - 1) / CONV_CHUNK, B), g2((C + 255) / 256, B);
+  if (B > 65535) throw std::runtime_error("sglb causal_conv1d: at most 65535 requests");
   using bf = __nv_bfloat16;
-  if (bf16) {
-    if (u_bf16)
-      causal_conv1d_fwd_kernel<bf, bf><<<g1, 256, 0, stream>>>((const bf*)x, ldx, (const bf*)w, (const bf*)bias, (const bf*)conv_state, cu_q, req_slots, seq_lens, C,
-                                                               K, silu ? 1 : 0, (bf*)u, ldu);
-    else
-      causal_conv1d_fwd_kernel<bf, float><<<g1, 256, 0, stream>>>((const bf*)x, ldx, (const bf*)w, (const bf*)bias, (const bf*)conv_state, cu_q, req_slots,
-                                                                  seq_lens, C, K, silu ? 1 : 0, (float*)u, ldu);
-    causal_conv1d_state_kernel<bf><<<g2, 256, 0, stream>>>((const bf*)x, ldx, (bf*)conv_state, cu_q, req_slots, seq_lens, C, K);
-  } else {
-    causal_conv1d_fwd_kernel<float, float><<<g1, 256, 0, stream>>>((const float*)x, ldx, (const float*)w, (const float*)bias, (const float*)conv_state, cu_q,
-                                                                   req_slots, seq_lens, C, K, silu ? 1 : 0, (float*)u, ldu);
-    causal_conv1d_state_kernel<float><<<g2, 256, 0, stream>>>((const float*)x, ldx, (float*)conv_state, cu_q, req_slots, seq_lens, C, K);
-  }
-  SGLB_CUDA_CHECK(cudaGetLastError());
+  if (bf16 && u_bf16) dispatch_conv1d<bf, bf>(x, ldx, w, bias, conv_state, cu_q, req_slots, seq_lens, B, max_q_len, C, K, silu, u, ldu, stream);
+  else if (bf16) dispatch_conv1d<bf, float>(x, ldx, w, bias, conv_state, cu_q, req_slots, seq_lens, B, max_q_len, C, K, silu, u, ldu, stream);
+  else dispatch_conv1d<float, float>(x, ldx, w, bias, conv_state, cu_q, req_slots, seq_lens, B, max_q_len, C, K, silu, u, ldu, stream);
 }
 
 // one warp per (b, h, p) state row of N floats; x / B / C / dt fp32 (already activated), state fp32 [slots, H, P, N]

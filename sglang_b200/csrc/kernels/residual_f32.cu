@@ -266,9 +266,10 @@ __global__ void __launch_bounds__(256) norm_add_f32_kernel(float* __restrict__ x
   }
 }
 
-// gate activations of grouped_rmsnorm
+// gate activations of grouped_rmsnorm; bf16 gates take the fast exponential and reciprocal (a few 2^-23 relative)
+template <typename TO>
 __device__ __forceinline__ float gate_act(float g, int silu) {
-  const float s = 1.f / (1.f + expf(-g));
+  const float s = sizeof(TO) == 2 ? __fdividef(1.f, 1.f + __expf(-g)) : 1.f / (1.f + expf(-g));
   return silu ? g * s : s;
 }
 
@@ -291,7 +292,7 @@ __global__ void __launch_bounds__(256) grouped_rmsnorm_kernel(const float* __res
   for (int i = threadIdx.x; i < per; i += 256) {
     float v = x[base + i] * rs;
     if (w) v *= ldf<TO>(w + c0 + i);
-    if (gr) v *= gate_act(ldf<TO>(gr + i), silu);
+    if (gr) v *= gate_act<TO>(ldf<TO>(gr + i), silu);
     stf<TO>(o + i, v);
   }
 }
@@ -307,11 +308,14 @@ __global__ void __launch_bounds__(256) grouped_rmsnorm_warp_kernel(const float* 
   const int n4 = per / 4;
   for (int g = warp; g < groups; g += 8) {
     const float4* xv = reinterpret_cast<const float4*>(x + (size_t)blockIdx.x * C + (size_t)g * per);
-    float4 keep[KEEP];
+    const size_t c0 = (size_t)g * per;
+    const TO* gr = gate ? gate + (size_t)blockIdx.x * ldg + c0 : nullptr;
+    float4 keep[KEEP], gk[KEEP];
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
       const int i = lane + k * 32;
+      gk[k] = gr && i < n4 ? ld4f<TO>(gr + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
       keep[k] = i < n4 ? xv[i] : make_float4(0.f, 0.f, 0.f, 0.f);
       ss += keep[k].x * keep[k].x + keep[k].y * keep[k].y + keep[k].z * keep[k].z + keep[k].w * keep[k].w;
     }
@@ -320,25 +324,23 @@ __global__ void __launch_bounds__(256) grouped_rmsnorm_warp_kernel(const float* 
       ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
     const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)per + eps) * out_scale;
-    const size_t c0 = (size_t)g * per;
-    auto emit = [&](int i, float4 v) {
+    auto emit = [&](int i, float4 v, float4 a) {
       v.x *= rs; v.y *= rs; v.z *= rs; v.w *= rs;
       if (w) {
-        const float4 a = ld4f<TO>(w + c0 + 4 * i);
-        v.x *= a.x; v.y *= a.y; v.z *= a.z; v.w *= a.w;
+        const float4 ww = ld4f<TO>(w + c0 + 4 * i);
+        v.x *= ww.x; v.y *= ww.y; v.z *= ww.z; v.w *= ww.w;
       }
-      if (gate) {
-        const float4 a = ld4f<TO>(gate + (size_t)blockIdx.x * ldg + c0 + 4 * i);
-        v.x *= gate_act(a.x, silu); v.y *= gate_act(a.y, silu); v.z *= gate_act(a.z, silu); v.w *= gate_act(a.w, silu);
+      if (gr) {
+        v.x *= gate_act<TO>(a.x, silu); v.y *= gate_act<TO>(a.y, silu); v.z *= gate_act<TO>(a.z, silu); v.w *= gate_act<TO>(a.w, silu);
       }
       st4f<TO>(out + (size_t)blockIdx.x * ldo + c0 + 4 * i, v);
     };
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
       const int i = lane + k * 32;
-      if (i < n4) emit(i, keep[k]);
+      if (i < n4) emit(i, keep[k], gk[k]);
     }
-    for (int i = lane + KEEP * 32; i < n4; i += 32) emit(i, xv[i]);
+    for (int i = lane + KEEP * 32; i < n4; i += 32) emit(i, xv[i], gr ? ld4f<TO>(gr + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
   }
 }
 

@@ -467,12 +467,20 @@ struct PrepParams {
 
 template <typename T>
 __global__ void __launch_bounds__(128) attention_prepare_kernel(const PrepParams p) {
+  extern __shared__ float2 trig[];              // (cos, sin) of the token's angles, computed once for all heads
   __shared__ float red[8];
   const int t = blockIdx.x;
   const int tid = threadIdx.x;
   const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
   const size_t slot = (size_t)p.loc[t];
   const int nq = p.H * p.D, nk = p.G * p.D;
+  const float pos = (float)p.positions[t];
+  const int half = p.inv_freq ? p.half : 0;
+  for (int m = tid; m < half; m += 128) {
+    float sn, cs;
+    sincosf(pos * p.inv_freq[m], &sn, &cs);
+    trig[m] = make_float2(cs, sn);
+  }
   float rq = 1.f, rk = 1.f;
   if (p.qw) {                                   // mean of squares over the whole q projection, then the whole k projection
     float sq = 0.f, sk = 0.f;
@@ -484,13 +492,12 @@ __global__ void __launch_bounds__(128) attention_prepare_kernel(const PrepParams
     rq = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)nq + p.eps);
     rk = 1.0f / sqrtf((red[4] + red[5] + red[6] + red[7]) / (float)nk + p.eps);
   }
-  const float pos = (float)p.positions[t];
+  if (!p.qw && half > 0) __syncthreads();
   const T* qw = reinterpret_cast<const T*>(p.qw);
   const T* kw = reinterpret_cast<const T*>(p.kw);
   T* qo = reinterpret_cast<T*>(p.q_out) + (size_t)t * p.H * p.Dq;
   T* ko = reinterpret_cast<T*>(p.kc) + slot * p.ldc;
   T* vo = reinterpret_cast<T*>(p.vc) + slot * p.ldc;
-  const int half = p.inv_freq ? p.half : 0;
   // q heads then k heads: element (head, i) of the padded destination
   const int total = p.H * p.Dq + p.G * p.hsk;
   for (int idx = tid; idx < total; idx += 128) {
@@ -508,8 +515,7 @@ __global__ void __launch_bounds__(128) attention_prepare_kernel(const PrepParams
     if (i < 2 * half) {
       const bool first = p.inter ? (i & 1) == 0 : i < half;
       const int fi = p.inter ? i >> 1 : first ? i : i - half;
-      float sn, cs;
-      sincosf(pos * p.inv_freq[fi], &sn, &cs);
+      const float cs = trig[fi].x, sn = trig[fi].y;
       const float other = val(p.inter ? i ^ 1 : first ? i + half : i - half);
       v = first ? v * cs - other * sn : v * cs + other * sn;
     }
@@ -554,12 +560,20 @@ __device__ __forceinline__ void wa_st2(__nv_bfloat16* p, float a, float b) { *re
 // two unrotated columns (or zero padding).
 template <typename T>
 __global__ void __launch_bounds__(128) attention_prepare_vec_kernel(const PrepParams p) {
+  extern __shared__ float2 trig[];              // (cos, sin) of the token's angles, computed once for all heads
   __shared__ float red[8];
   const int t = blockIdx.x;
   const int tid = threadIdx.x;
   const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
   const size_t slot = (size_t)p.loc[t];
   const int nq = p.H * p.D, nk = p.G * p.D;
+  const float pos = (float)p.positions[t];
+  const int half = p.inv_freq ? p.half : 0;
+  for (int m = tid; m < half; m += 128) {
+    float sn, cs;
+    sincosf(pos * p.inv_freq[m], &sn, &cs);
+    trig[m] = make_float2(cs, sn);
+  }
   float rq = 1.f, rk = 1.f;
   if (p.qw) {
     float sq = 0.f, sk = 0.f;
@@ -571,48 +585,45 @@ __global__ void __launch_bounds__(128) attention_prepare_vec_kernel(const PrepPa
     rq = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)nq + p.eps);
     rk = 1.0f / sqrtf((red[4] + red[5] + red[6] + red[7]) / (float)nk + p.eps);
   }
-  const float pos = (float)p.positions[t];
+  if (!p.qw && half > 0) __syncthreads();
   const T* qw = reinterpret_cast<const T*>(p.qw);
   const T* kw = reinterpret_cast<const T*>(p.kw);
   T* qo = reinterpret_cast<T*>(p.q_out) + (size_t)t * p.H * p.Dq;
   T* ko = reinterpret_cast<T*>(p.kc) + slot * p.ldc;
   T* vo = reinterpret_cast<T*>(p.vc) + slot * p.ldc;
-  const int half = p.inv_freq ? p.half : 0;
   const int nrot = p.inter ? half : half / 2;             // rotated items per head
   const int per_q = nrot + (p.Dq - 2 * half) / 2, per_k = nrot + (p.hsk - 2 * half) / 2;
-  const int total = p.H * per_q + p.G * per_k;
-  for (int idx = tid; idx < total; idx += 128) {
-    const bool isq = idx < p.H * per_q;
-    const int rel = isq ? idx : idx - p.H * per_q;
-    const int per = isq ? per_q : per_k, hs = isq ? p.Dq : p.hsk;
-    const int hd = rel / per, it = rel - hd * per;
+  // a warp takes a head at a time
+  for (int hh = tid >> 5; hh < p.H + p.G; hh += 4) {
+    const bool isq = hh < p.H;
+    const int hd = isq ? hh : hh - p.H;
+    const int per = isq ? per_q : per_k;
     const T* src = row + (isq ? 0 : nq) + hd * p.D;
     const T* w = isq ? qw : kw;
     const float r = isq ? rq : rk;
-    T* dst = (isq ? qo : ko) + (size_t)hd * hs;
+    T* dst = isq ? qo + (size_t)hd * p.Dq : ko + (size_t)hd * p.hsk;
     auto val2 = [&](int c) {
       float2 v = wa_ld2(src + c);
       v.x *= r; v.y *= r;
       if (w) { const float2 ww = wa_ld2(w + hd * p.D + c); v.x *= ww.x; v.y *= ww.y; }
       return v;
     };
-    if (it < nrot && p.inter) {
-      const float2 a = val2(2 * it);
-      float sn, cs;
-      sincosf(pos * p.inv_freq[it], &sn, &cs);
-      wa_st2(dst + 2 * it, a.x * cs - a.y * sn, a.y * cs + a.x * sn);
-    } else if (it < nrot) {
-      const int i = 2 * it;
-      const float2 a = val2(i), b = val2(i + half);
-      float s0, c0, s1, c1;
-      sincosf(pos * p.inv_freq[i], &s0, &c0);
-      sincosf(pos * p.inv_freq[i + 1], &s1, &c1);
-      wa_st2(dst + i, a.x * c0 - b.x * s0, a.y * c1 - b.y * s1);
-      wa_st2(dst + i + half, b.x * c0 + a.x * s0, b.y * c1 + a.y * s1);
-    } else {
-      const int c = 2 * half + 2 * (it - nrot);
-      if (c < p.D) { const float2 v = val2(c); wa_st2(dst + c, v.x, v.y); }
-      else wa_st2(dst + c, 0.f, 0.f);
+    for (int it = tid & 31; it < per; it += 32) {
+      if (it < nrot && p.inter) {
+        const float2 a = val2(2 * it);
+        const float cs = trig[it].x, sn = trig[it].y;
+        wa_st2(dst + 2 * it, a.x * cs - a.y * sn, a.y * cs + a.x * sn);
+      } else if (it < nrot) {
+        const int i = 2 * it;
+        const float2 a = val2(i), b = val2(i + half);
+        const float c0 = trig[i].x, s0 = trig[i].y, c1 = trig[i + 1].x, s1 = trig[i + 1].y;
+        wa_st2(dst + i, a.x * c0 - b.x * s0, a.y * c1 - b.y * s1);
+        wa_st2(dst + i + half, b.x * c0 + a.x * s0, b.y * c1 + a.y * s1);
+      } else {
+        const int c = 2 * half + 2 * (it - nrot);
+        if (c < p.D) { const float2 v = val2(c); wa_st2(dst + c, v.x, v.y); }
+        else wa_st2(dst + c, 0.f, 0.f);
+      }
     }
   }
   const T* vs = row + nq + nk;
@@ -678,12 +689,14 @@ void attention_prepare(const void* qkv, int ld, bool bf16, int T, int H, int G, 
   auto al = [&](const void* q) { return q == nullptr || ((uintptr_t)q % a2) == 0; };
   const bool vec = D % 2 == 0 && Dv % 2 == 0 && (interleaved || half % 2 == 0) && ld % 2 == 0 && ldc % 2 == 0 && p.Dq % 2 == 0 && p.hsk % 2 == 0 && p.hsv % 2 == 0 &&
                    (v_inv_freq == nullptr || v_interleaved || Dv % 4 == 0) && (v_first == nullptr || ldvf % 2 == 0) && al(qkv) && al(kc) && al(vc) && al(q_out) && al(v_first) && al(q_norm_w) && al(k_norm_w);
+  const size_t smem = inv_freq ? sizeof(float2) * (size_t)half : 0;
+  if (smem > 40 * 1024) throw std::runtime_error("sglb attention_prepare: rotary widths up to 10,240");
   if (vec) {
-    if (bf16) attention_prepare_vec_kernel<__nv_bfloat16><<<T, 128, 0, stream>>>(p);
-    else attention_prepare_vec_kernel<float><<<T, 128, 0, stream>>>(p);
+    if (bf16) attention_prepare_vec_kernel<__nv_bfloat16><<<T, 128, smem, stream>>>(p);
+    else attention_prepare_vec_kernel<float><<<T, 128, smem, stream>>>(p);
   } else {
-    if (bf16) attention_prepare_kernel<__nv_bfloat16><<<T, 128, 0, stream>>>(p);
-    else attention_prepare_kernel<float><<<T, 128, 0, stream>>>(p);
+    if (bf16) attention_prepare_kernel<__nv_bfloat16><<<T, 128, smem, stream>>>(p);
+    else attention_prepare_kernel<float><<<T, 128, smem, stream>>>(p);
   }
   SGLB_CUDA_CHECK(cudaGetLastError());
 }
