@@ -28,6 +28,55 @@ __device__ __forceinline__ float tanh_by_exp(float z) {
   return 1.f - __fdividef(2.f, t + 1.f);
 }
 
+// tanh(z) / z as a polynomial in t = z^2 on [0, 1] (Chebyshev interpolation of degree 7, rounded to fp32): relative error of tanh about 1e-7
+__device__ __forceinline__ float tanh_ratio(float t) {
+  float p = fmaf(t, -0.00035232809f, 0.0022786476f);
+  p = fmaf(t, p, -0.007912485f);
+  p = fmaf(t, p, 0.02146141f);
+  p = fmaf(t, p, -0.053869706f);
+  p = fmaf(t, p, 0.13332139f);
+  p = fmaf(t, p, -0.33333278f);
+  return fmaf(t, p, 1.f);
+}
+
+// score cap and distance bias on a row of raw scores (so that raw * scale is the final logit).  Where all 32 rows of the warp stay within the cap
+// (the usual case: caps are meant for outliers) the cap is a polynomial on the multiply-add pipe, which has room beside the soft-max's
+// exponentials; otherwise it is formed with the special-function instructions, which do not.
+template <int NC>
+__device__ __forceinline__ void cap_and_bias(uint32_t (&sr)[NC][32], float cap, float inv_cap, float scale_nat, float inv_scale_nat, bool biased, float slope,
+                                             float off) {
+  if (cap > 0.f) {
+    const float k = scale_nat * inv_cap;
+    float mx = 0.f;
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+      for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fabsf(__uint_as_float(sr[c][i])));
+    if (!__any_sync(0xffffffffu, mx * k > 1.f)) {
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float x = __uint_as_float(sr[c][i]), z = x * k;
+          sr[c][i] = __float_as_uint(x * tanh_ratio(z * z));
+        }
+    } else {
+      const float back = cap * inv_scale_nat;
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(back * tanh_by_exp(__uint_as_float(sr[c][i]) * k));
+    }
+  }
+  if (biased) {
+    const float sl = slope * inv_scale_nat, of = off * inv_scale_nat;
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+      for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(fmaf(sl, (float)(c * 32 + i), __uint_as_float(sr[c][i]) + of));
+  }
+}
+
 constexpr int ATT_D = 128;          // head dim
 // kv tile KT is a template parameter: 128 for prefill (compute-bound, 1 CTA/SM), 64 for decode (latency-bound: 256
 // TMEM columns + 96 KB smem so two CTAs share an SM and overlap their load -> MMA -> softmax chains)
@@ -324,15 +373,8 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
               sr[c][i] = __float_as_uint(fmaf(-log_coef, __log2f(fmaf(rate, dist, 1.f)), __uint_as_float(sr[c][i])));
             }
         } else if (HAS_CAP) {   // soft-capping and / or distance bias (separate template instance): rewrite raw so raw*scale_log2 is the final logit
-          const float off = -slope * (float)(q_pos - kv0);      // bias of column 0; column c adds slope * c
-#pragma unroll
-          for (int c = 0; c < NC; ++c)
-#pragma unroll
-            for (int i = 0; i < 32; ++i) {
-              const float x = __uint_as_float(sr[c][i]) * scale_nat;
-              const float y = cap > 0.f ? cap * tanh_by_exp(x * inv_cap) : x;
-              sr[c][i] = __float_as_uint(fmaf(slope, (float)(c * 32 + i), y + off) * inv_scale_nat);
-            }
+          // bias of column 0; column c adds slope * c
+          cap_and_bias<NC>(sr, cap, inv_cap, scale_nat, inv_scale_nat, p.slopes != nullptr, slope, -slope * (float)(q_pos - kv0));
         }
         float mx_raw = -INFINITY;
         if (need_mask) {
@@ -747,15 +789,8 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
                 sr[c][i] = __float_as_uint(fmaf(-log_coef, __log2f(fmaf(rate, dist, 1.f)), __uint_as_float(sr[c][i])));
               }
           } else if (HAS_CAP) {
-            const float off = -slope * (float)(q_pos - kv0);
-#pragma unroll
-            for (int c = 0; c < NC; ++c)
-#pragma unroll
-              for (int i = 0; i < 32; ++i) {
-                const float x = __uint_as_float(sr[c][i]) * scale_nat;
-                const float y = cap > 0.f ? cap * tanh_by_exp(x * inv_cap) : x;
-                sr[c][i] = __float_as_uint(fmaf(slope, (float)(c * 32 + i), y + off) * inv_scale_nat);
-              }
+            // bias of column 0; column c adds slope * c
+            cap_and_bias<NC>(sr, cap, inv_cap, scale_nat, inv_scale_nat, p.slopes != nullptr, slope, -slope * (float)(q_pos - kv0));
           }
           float mx_raw = -INFINITY;
           if (need_mask) {

@@ -298,12 +298,11 @@ __global__ void __launch_bounds__(256) grouped_rmsnorm_kernel(const float* __res
 }
 
 // the same with one warp per (row, part): a CTA of 8 warps walks the parts of its row (many small parts: no CTA-wide barrier, four columns per
-// access); a part of up to 512 columns stays in registers between the two passes
-template <typename TO>
+// access); a part of up to KEEP * 128 columns stays in registers between the two passes
+template <typename TO, int KEEP>
 __global__ void __launch_bounds__(256) grouped_rmsnorm_warp_kernel(const float* __restrict__ x, const TO* __restrict__ w, TO* __restrict__ out, int C,
                                                                    int per, int groups, float eps, const TO* __restrict__ gate, int ldg, int ldo,
                                                                    float out_scale, int silu) {
-  constexpr int KEEP = 4;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n4 = per / 4;
   for (int g = warp; g < groups; g += 8) {
@@ -610,8 +609,11 @@ void grouped_rmsnorm(const float* x, const void* w, void* out, bool out_bf16, in
   auto al = [&](const void* p) { return p == nullptr || ((uintptr_t)p % a4) == 0; };
   using bf = __nv_bfloat16;
   if (groups >= 4 && per % 4 == 0 && per <= 4096 && ldo % 4 == 0 && (!gate || ldg % 4 == 0) && ((uintptr_t)x % 16) == 0 && al(w) && al(out) && al(gate)) {
-    if (out_bf16) grouped_rmsnorm_warp_kernel<bf><<<T, 256, 0, stream>>>(x, (const bf*)w, (bf*)out, C, per, groups, eps, (const bf*)gate, ldg, ldo, out_scale, act);
-    else grouped_rmsnorm_warp_kernel<float><<<T, 256, 0, stream>>>(x, (const float*)w, (float*)out, C, per, groups, eps, (const float*)gate, ldg, ldo, out_scale, act);
+#define SGLB_GN(TO, KEEP) \
+  grouped_rmsnorm_warp_kernel<TO, KEEP><<<T, 256, 0, stream>>>(x, (const TO*)w, (TO*)out, C, per, groups, eps, (const TO*)gate, ldg, ldo, out_scale, act)
+    if (out_bf16) { if (per <= 128) SGLB_GN(bf, 1); else if (per <= 256) SGLB_GN(bf, 2); else SGLB_GN(bf, 4); }
+    else { if (per <= 128) SGLB_GN(float, 1); else if (per <= 256) SGLB_GN(float, 2); else SGLB_GN(float, 4); }
+#undef SGLB_GN
     SGLB_CUDA_CHECK(cudaGetLastError());
     return;
   }

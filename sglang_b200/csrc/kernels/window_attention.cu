@@ -366,6 +366,31 @@ __global__ void __launch_bounds__(128) sigmoid_gate_kernel(const T* __restrict__
   }
 }
 
+// the same with 16-byte accesses: one CTA per token walks its heads in groups of eight (bf16) or four (fp32) columns
+template <typename T>
+__global__ void __launch_bounds__(256) sigmoid_gate_vec_kernel(const T* __restrict__ o, int hs, const T* __restrict__ gate, int ldg, int per_head, int H, int Dv,
+                                                               float scale, T* __restrict__ out, int ldo) {
+  constexpr int V = 16 / sizeof(T);
+  const int per = Dv / V, total = H * per;
+  const T* src = o + (size_t)blockIdx.x * H * hs;
+  const T* g = gate + (size_t)blockIdx.x * ldg;
+  T* dst = out + (size_t)blockIdx.x * ldo;
+  auto sig = [](float x) { return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-x)) : 1.f / (1.f + expf(-x)); };
+  for (int idx = threadIdx.x; idx < total; idx += 256) {
+    const int h = idx / per, c = (idx - h * per) * V;
+    const uint4 raw = *reinterpret_cast<const uint4*>(src + (size_t)h * hs + c);
+    const T* v = reinterpret_cast<const T*>(&raw);
+    uint4 graw = make_uint4(0, 0, 0, 0), oraw;
+    if (!per_head) graw = *reinterpret_cast<const uint4*>(g + (size_t)h * Dv + c);
+    const T* gv = reinterpret_cast<const T*>(&graw);
+    T* ov = reinterpret_cast<T*>(&oraw);
+    const float gh = per_head ? scale * sig(wa_ld<T>(g + h)) : 0.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) wa_st<T>(ov + e, wa_ld<T>(v + e) * (per_head ? gh : scale * sig(wa_ld<T>(gv + e))));
+    *reinterpret_cast<uint4*>(dst + (size_t)h * Dv + c) = oraw;
+  }
+}
+
 // out[t, h * Dv + c] = the head o[t, h, :Dv] (rows of hs elements) times sigmoid(lse[t, h] - sink[h]) (lse null: times 1), turned over its whole
 // width by -+ position * inv_freq[m]: pair m = columns (m, m + Dv/2) or, inter, (2m, 2m + 1).  Angle, sine and cosine fp32.  One CTA per token:
 // a thread owns a pair index and walks the heads, so that the sine and cosine of an angle are computed once for all heads.
@@ -667,6 +692,17 @@ __global__ void __launch_bounds__(128) attention_prepare_vec_kernel(const PrepPa
 void sigmoid_gate(const void* o, int head_stride, const void* gate, int ldg, bool per_head, bool bf16, int T, int H, int Dv, float scale, void* out, int ldo,
                   cudaStream_t stream) {
   if (T <= 0 || H <= 0) return;
+  const int v = bf16 ? 8 : 4;
+  auto al = [](const void* p) { return (uintptr_t)p % 16 == 0; };
+  if (Dv % v == 0 && head_stride % v == 0 && ldo % v == 0 && al(o) && al(out) && (per_head || (ldg % v == 0 && al(gate)))) {
+    if (bf16)
+      sigmoid_gate_vec_kernel<__nv_bfloat16><<<T, 256, 0, stream>>>((const __nv_bfloat16*)o, head_stride, (const __nv_bfloat16*)gate, ldg, per_head ? 1 : 0, H, Dv,
+                                                                    scale, (__nv_bfloat16*)out, ldo);
+    else
+      sigmoid_gate_vec_kernel<float><<<T, 256, 0, stream>>>((const float*)o, head_stride, (const float*)gate, ldg, per_head ? 1 : 0, H, Dv, scale, (float*)out, ldo);
+    SGLB_CUDA_CHECK(cudaGetLastError());
+    return;
+  }
   if (bf16)
     sigmoid_gate_kernel<__nv_bfloat16><<<T * H, 128, 0, stream>>>((const __nv_bfloat16*)o, head_stride, (const __nv_bfloat16*)gate, ldg, per_head ? 1 : 0, H, Dv,
                                                                   scale, (__nv_bfloat16*)out, ldo);

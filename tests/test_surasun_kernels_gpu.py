@@ -208,6 +208,49 @@ def test_gated_recurrence_at_the_ends_of_its_range(dtype):
     torch.testing.assert_close(got.cpu().float(), ref, **_tol(dtype, f32=(3e-4, 5e-4), bf=(8e-3, 1e-2)))
 
 
+@pytest.mark.parametrize("outliers", [False, True])
+@pytest.mark.parametrize("decode", [False, True])
+def test_score_cap_on_the_tensor_core_kernels(decode, outliers):
+    """scores that stay within the cap, and a few far beyond it in some rows only: both forms of the cap, in prompt tiles and in decode"""
+    _need()
+    g = torch.Generator().manual_seed(7)
+    H, G, D, ps, cap = 8, 2, 128, 64, 9.0
+    lens, cached = ([1] * 5, [130, 0, 400, 63, 64]) if decode else ([70, 1, 300, 64], [0, 99, 31, 200])
+    tot = [a + b for a, b in zip(lens, cached)]
+    per = (max(tot) + ps - 1) // ps
+    pt = (torch.randperm(len(lens) * per, generator=g).int() + 1).view(len(lens), per)
+    kc, vc = (torch.randn((len(lens) * per + 2) * ps, G, D, generator=g).bfloat16() for _ in range(2))
+    q = torch.randn(sum(lens), H, D, generator=g)
+    if outliers:
+        q[::37] *= 12.0
+    q = q.bfloat16()
+    rows, sl, ql = _i32(list(range(len(lens))), "cpu"), _i32(tot, "cpu"), _i32(lens, "cpu")
+    ref = torch_ref.window_attention(q.float(), kc.float().view(-1, 1, G * D), vc.float().view(-1, 1, G * D), G, D, pt, rows, sl, ql, ps, D ** -0.5, cap, -1, None, None, D)
+    cu = None if decode else _i32([0, *np.cumsum(lens).tolist()])
+    a = [t.to(DEV) for t in (q, kc, vc, pt, rows, sl, ql)]
+    assert ops.tc_attention_ok(a[0], a[1], a[2], ps)
+    for splits in ((1, 3) if decode else (1,)):
+        got = ops.paged_attention(a[0], a[1], a[2], a[3], a[4], a[5], cu, a[6], max(lens), ps, D ** -0.5, logit_cap=cap, num_splits=splits)
+        torch.testing.assert_close(got.cpu().float(), ref, rtol=3e-2, atol=2e-2)
+
+
+@BOTH
+@pytest.mark.parametrize("H,hs,Dv", [(3, 128, 48), (8, 64, 64), (5, 7, 7), (2, 128, 100)])
+def test_sigmoid_gate(H, hs, Dv, dtype):
+    _need()
+    g = torch.Generator().manual_seed(H)
+    T = 33
+    o, wide = torch.randn(T, H, hs, generator=g).to(dtype), torch.randn(T, H * Dv + 8, generator=g).to(dtype)
+    for gate in (wide[:, :H], wide[:, 8:], wide[:, 3:3 + H * Dv]):
+        ref = ops.sigmoid_gate(o, gate, Dv, 0.7)
+        buf = torch.full((T, H * Dv + 24), 5.0, dtype=dtype, device=DEV)
+        for at in (0, 8, 3):
+            at_gate = wide.to(DEV)[:, gate.storage_offset():gate.storage_offset() + gate.shape[1]]
+            ops.sigmoid_gate(o.to(DEV), at_gate, Dv, 0.7, buf[:, at:at + H * Dv])
+            torch.testing.assert_close(buf[:, at:at + H * Dv].cpu().float(), ref.float(), **_tol(dtype))
+        assert float(buf[:, 8 + H * Dv:].min()) == 5.0
+
+
 # ------------------------------------------------------------------ the engine
 def _spread_error(x, ref):
     """per position: root mean square of the difference over the vocabulary (mean taken off) against that of the logits"""
