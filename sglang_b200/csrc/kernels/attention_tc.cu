@@ -39,42 +39,34 @@ __device__ __forceinline__ float tanh_ratio(float t) {
   return fmaf(t, p, 1.f);
 }
 
-// score cap and distance bias on a row of raw scores (so that raw * scale is the final logit).  Where all 32 rows of the warp stay within the cap
-// (the usual case: caps are meant for outliers) the cap is a polynomial on the multiply-add pipe, which has room beside the soft-max's
-// exponentials; otherwise it is formed with the special-function instructions, which do not.
+// score cap on a row of raw scores in TMEM (so that raw * scale is the capped logit), 32 columns at a time and back to where they were: as a rolled
+// loop of its own it stays in the instruction cache, unlike one more 128-wide unrolled pass over the row in registers.  Where all 32 rows of the
+// warp stay within the cap (the usual case: caps are meant for outliers) the cap is a polynomial on the multiply-add pipe, which has room beside
+// the soft-max's exponentials; otherwise it is formed with the special-function instructions.
 template <int NC>
-__device__ __forceinline__ void cap_and_bias(uint32_t (&sr)[NC][32], float cap, float inv_cap, float scale_nat, float inv_scale_nat, bool biased, float slope,
-                                             float off) {
-  if (cap > 0.f) {
-    const float k = scale_nat * inv_cap;
+__device__ __forceinline__ void cap_scores(uint32_t s_addr, float cap, float inv_cap, float scale_nat, float inv_scale_nat) {
+  const float k = scale_nat * inv_cap, back = cap * inv_scale_nat;
+#pragma unroll 1
+  for (int c = 0; c < NC; ++c) {
+    uint32_t x[32];
+    tmem_ld_32x32b_x32(s_addr + c * 32, x);
+    tmem_ld_wait();
     float mx = 0.f;
 #pragma unroll
-    for (int c = 0; c < NC; ++c)
-#pragma unroll
-      for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fabsf(__uint_as_float(sr[c][i])));
+    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fabsf(__uint_as_float(x[i])));
     if (!__any_sync(0xffffffffu, mx * k > 1.f)) {
 #pragma unroll
-      for (int c = 0; c < NC; ++c)
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          const float x = __uint_as_float(sr[c][i]), z = x * k;
-          sr[c][i] = __float_as_uint(x * tanh_ratio(z * z));
-        }
+      for (int i = 0; i < 32; ++i) {
+        const float v = __uint_as_float(x[i]), z = v * k;
+        x[i] = __float_as_uint(v * tanh_ratio(z * z));
+      }
     } else {
-      const float back = cap * inv_scale_nat;
 #pragma unroll
-      for (int c = 0; c < NC; ++c)
-#pragma unroll
-        for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(back * tanh_by_exp(__uint_as_float(sr[c][i]) * k));
+      for (int i = 0; i < 32; ++i) x[i] = __float_as_uint(back * tanh_by_exp(__uint_as_float(x[i]) * k));
     }
+    tmem_st_32x32b_x32(s_addr + c * 32, x);
   }
-  if (biased) {
-    const float sl = slope * inv_scale_nat, of = off * inv_scale_nat;
-#pragma unroll
-    for (int c = 0; c < NC; ++c)
-#pragma unroll
-      for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(fmaf(sl, (float)(c * 32 + i), __uint_as_float(sr[c][i]) + of));
-  }
+  tmem_st_wait();
 }
 
 constexpr int ATT_D = 128;          // head dim
@@ -353,6 +345,7 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       if (warp_valid) {
         constexpr int NC = KT / 32;
         const uint32_t s_addr = tmem_S0 + lane_addr + st * KT;
+        if (HAS_CAP && cap > 0.f) cap_scores<NC>(s_addr, cap, inv_cap, scale_nat, inv_scale_nat);
         uint32_t sr[NC][32];
 #pragma unroll
         for (int c = 0; c < NC; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, sr[c]);
@@ -372,9 +365,12 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
               const float dist = fmaxf(d0 - (float)(c * 32 + i), 0.f);
               sr[c][i] = __float_as_uint(fmaf(-log_coef, __log2f(fmaf(rate, dist, 1.f)), __uint_as_float(sr[c][i])));
             }
-        } else if (HAS_CAP) {   // soft-capping and / or distance bias (separate template instance): rewrite raw so raw*scale_log2 is the final logit
-          // bias of column 0; column c adds slope * c
-          cap_and_bias<NC>(sr, cap, inv_cap, scale_nat, inv_scale_nat, p.slopes != nullptr, slope, -slope * (float)(q_pos - kv0));
+        } else if (HAS_CAP && p.slopes) {   // distance bias (separate template instance): rewrite raw so raw*scale_log2 is the final logit
+          const float sl = slope * inv_scale_nat, off = -sl * (float)(q_pos - kv0);      // bias of column 0; column c adds slope * c
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(fmaf(sl, (float)(c * 32 + i), __uint_as_float(sr[c][i]) + off));
         }
         float mx_raw = -INFINITY;
         if (need_mask) {
@@ -772,6 +768,7 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         if (warp_valid) {
           constexpr int NC = KT / 32;
           const uint32_t s_addr = tmem_S0 + lane_addr + st * KT;
+          if (HAS_CAP && cap > 0.f) cap_scores<NC>(s_addr, cap, inv_cap, scale_nat, inv_scale_nat);
           uint32_t sr[NC][32];
 #pragma unroll
           for (int c = 0; c < NC; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, sr[c]);
@@ -788,9 +785,12 @@ attn_fwd_tc_persist_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
                 const float dist = fmaxf(d0 - (float)(c * 32 + i), 0.f);
                 sr[c][i] = __float_as_uint(fmaf(-log_coef, __log2f(fmaf(rate, dist, 1.f)), __uint_as_float(sr[c][i])));
               }
-          } else if (HAS_CAP) {
-            // bias of column 0; column c adds slope * c
-            cap_and_bias<NC>(sr, cap, inv_cap, scale_nat, inv_scale_nat, p.slopes != nullptr, slope, -slope * (float)(q_pos - kv0));
+          } else if (HAS_CAP && p.slopes) {
+            const float sl = slope * inv_scale_nat, off = -sl * (float)(q_pos - kv0);      // bias of column 0; column c adds slope * c
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+#pragma unroll
+              for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(fmaf(sl, (float)(c * 32 + i), __uint_as_float(sr[c][i]) + off));
           }
           float mx_raw = -INFINITY;
           if (need_mask) {
