@@ -3,7 +3,7 @@
 
     u   = sum_s in[s] x_s
     y   = sublayer(norm(u))
-    x_t <- sum_s mix[s, t] x_s + mult * out[t] * y            all streams at once, from the old ones
+    x_t <- sum_s mix[s, t] x_s + mult * out[t] * y            simultaneously for every t
 
 The streams start as S copies of the embedding output and end as their sum.  ``ops.stream_mix_norm`` applies one sublayer's update, forms the
 next sublayer's u and norms it in one kernel over the fp32 streams; ``StreamMix.pack`` makes the numbers it takes.  With one stream and

@@ -1,4 +1,4 @@
-"""Gated linear recurrence block (Griffin's recurrent block with a real-gated linear recurrent unit):
+"""Gated linear recurrence block, the RG-LRU layer of Griffin-style models:
 
     y, x = W_y h + b_y, W_x h + b_x                      one GEMM, rows [y | x]
     u    = causal convolution of x per channel (+ bias, no activation)
